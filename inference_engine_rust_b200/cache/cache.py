@@ -7,7 +7,8 @@ sequence and appends at `current_pos` (src/layers/attention.rs:16-74); a window 
 mask over that full-length buffer (:610-613).  Here memory is counted in pages of
 `page_tokens` positions shared by all live sequences, each sequence has its own length, and
 a windowed group keeps only `ceil(window / page_tokens)` pages per sequence, written round
-and round.  Because keys are rotated before they are stored, where a key lies in the ring
+and round; first positions that stay visible behind a window keep pages of their own in front of
+that ring.  Because keys are rotated before they are stored, where a key lies in the ring
 does not matter to the result.
 """
 from __future__ import annotations
@@ -32,6 +33,7 @@ class KVRequest:
     window: Optional[int] = None     # None: every earlier key stays visible
     values: bool = True              # False: one row per position (keys only), e.g. a shared latent
     chunk: Optional[int] = None      # C: a position sees only its own chunk of C positions (counted from position 0)
+    keep: int = 0                    # the first `keep` positions of a sequence stay visible whatever window and chunk say
 
     @property
     def reach(self) -> Optional[int]:
@@ -65,10 +67,14 @@ class KVGroup:
         self.dtype = dtype
         self.device = device
         self.table_width = max(1, math.ceil(max_seq_len / page_tokens))
+        self.keep_pages = 0          # pages in front of the ring that stay: those of the kept first positions
         if req.reach is None:
             self.ring_pages = self.table_width
         else:
-            self.ring_pages = min(self.table_width, max(1, math.ceil(req.reach / page_tokens)))
+            keep_pages = math.ceil(req.keep / page_tokens)
+            self.ring_pages = min(self.table_width, keep_pages + max(1, math.ceil(req.reach / page_tokens)))
+            if self.ring_pages < self.table_width:
+                self.keep_pages = keep_pages
         shape = (len(self.layers), n_pages, req.kv_heads, page_tokens, req.head_dim)
         self.k = torch.empty(shape, dtype=dtype, device=device)
         self.v = torch.empty(shape if req.values else (len(self.layers), 0) + shape[2:], dtype=dtype, device=device)
@@ -84,7 +90,8 @@ class KVGroup:
 
     @property
     def ring_capacity(self) -> int:
-        return self.ring_pages * self.page_tokens
+        """The latest positions that are certain to be held (kept first positions apart)."""
+        return (self.ring_pages - self.keep_pages) * self.page_tokens
 
     def pages_needed(self, length: int) -> int:
         return min(self.ring_pages, math.ceil(length / self.page_tokens))
@@ -246,7 +253,8 @@ class Cache:
         return B.KvView(k=g.k[i].data_ptr(), v=g.v[i].data_ptr() if g.req.values else None, page_table=g.table.data_ptr(),
                         table_width=g.table_width, ring_pages=g.ring_pages, page_tokens=g.page_tokens,
                         n_pages=g.n_pages, kv_heads=g.req.kv_heads, head_dim=g.req.head_dim,
-                        dtype=B.dtype_code(g.dtype), window=g.req.window or 0, chunk=g.req.chunk or 0)
+                        dtype=B.dtype_code(g.dtype), window=g.req.window or 0, chunk=g.req.chunk or 0,
+                        keep=g.req.keep if g.req.reach is not None else 0, keep_pages=g.keep_pages)
 
     # ---- slots ------------------------------------------------------------------------
     def open_sequence(self) -> int:
@@ -304,7 +312,7 @@ class Cache:
             for s in slots:
                 n = int(self.seq_lens[s])
                 if g.req.reach is not None:
-                    n = min(n, g.req.reach)
+                    n = min(n, g.req.reach + g.req.keep)
                 total += n * g.bytes_per_token()
         return total
 

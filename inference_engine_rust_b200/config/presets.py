@@ -141,6 +141,36 @@ PRESETS["vufinex-12b-sizes"] = _vufinex(5120, 131072, 40, 32, 8, 128, 8192, 80, 
 PRESETS["vufinex-tiny"] = _vufinex(96, 320, 8, 4, 2, 16, 24, 3, 32, 8, 16, 8, 24, 40, 6, 2, 3, 2, 32, shared_from=4)
 
 
+def _botulorn(width, vocab, layers, heads, kv_heads, dim, vdim, window, keep, lat_dim, rot_dim, lat_vdim, q_rank, kv_rank, lat_window,
+              ff, buckets, original, factor=4.0):
+    """A Botulorn configuration whose layers go round latent attention, attention, attention, latent attention, each with a
+    dense feed-forward; all attention layers mix values."""
+    stretch = {"factor": factor, "original": original, "fast": 32.0, "slow": 1.0}
+    mixers = [
+        ("latent_attention", {"heads": heads, "dim": lat_dim, "rot_dim": rot_dim, "vdim": lat_vdim, "q_rank": q_rank, "kv_rank": kv_rank,
+                              "scale": (lat_dim + rot_dim) ** -0.5, "mask": {"size": lat_window},
+                              "rot": {"base": 500000.0, "dims": rot_dim, "scaling": dict(stretch)}}),
+        ("attention", {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
+                       "mask": {"size": window, "keep_first": keep}, "v_mix": True,
+                       "rot": {"base": 10000.0, "dims": dim, "scaling": dict(stretch)}}),
+    ]
+    out = []
+    for i in range(layers):
+        kind, mixer = mixers[0 if i % 4 in (0, 3) else 1]
+        out.append({"type": kind, "mixer": copy.deepcopy(mixer), "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Botulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 8.0, "bigram": {"buckets": buckets, "mul_prev": 1009, "mul_cur": 31}}, "layers": out}
+
+
+# Botulorn at the width, head count, head size and feed-forward size of Mistral 7B (latent attention with 128 unrotated and 64
+# rotated numbers per head over latents of 1,536 and 512; windows of 4,096 positions, the first four kept), and a tiny one that
+# runs anywhere in seconds.
+PRESETS["botulorn-7b-sizes"] = _botulorn(4096, 32000, 32, 32, 8, 128, 128, 4096, 4, 128, 64, 128, 1536, 512, 4096, 14336, 65521, 4096)
+# the same at the sizes of Mistral NeMo 12B (width 5,120, a vocabulary of 131,072)
+PRESETS["botulorn-12b-sizes"] = _botulorn(5120, 131072, 40, 32, 8, 128, 128, 4096, 4, 128, 64, 128, 1536, 512, 4096, 14336, 65521, 4096)
+PRESETS["botulorn-tiny"] = _botulorn(80, 320, 4, 6, 3, 16, 24, 20, 2, 12, 8, 16, 24, 40, 28, 72, 101, 64)
+
+
 def preset(name: str) -> dict:
     """A copy of the named configuration (a config.json-style dict)."""
     try:

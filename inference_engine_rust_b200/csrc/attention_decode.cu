@@ -95,7 +95,7 @@ attention_decode_kernel(DecodeParams p, IertBatchView b, IertKvView c) {
 
   for (int blk = my_lo + warp; blk < my_hi; blk += WARPS) {
     const int lblk = blk / blocks_per_page;                       // logical page of the sequence
-    const int page = c.page_table[(size_t)slot * c.table_width + lblk % c.ring_pages];
+    const int page = c.page_table[(size_t)slot * c.table_width + iert_table_entry(c, lblk)];
     if (page < 0 || page >= c.n_pages) {
       if (lane == 0) atomicOr(p.err, IERT_ERR_PAGE_RANGE);
       continue;
@@ -252,14 +252,14 @@ IERT_API long long iert_attention_decode_scratch_floats(int n_tokens, int heads,
 // qkv: packed bf16 projection of the step (one token per sequence), queries rotated, the new
 // keys and values already stored in the cache.  out: bf16 [T, heads * head_dim].
 // scratch: iert_attention_decode_scratch_floats(...) floats.  splits >= 1.
-// Takes bf16 caches with head_dim a multiple of 8 up to 256 and page_tokens a multiple of 32;
+// Takes bf16 caches with head_dim a multiple of 8 up to 256, page_tokens a multiple of 32 and no kept first positions;
 // anything else returns IERT_BAD_ARGUMENT and launches nothing.
 IERT_API int iert_attention_decode(const void* qkv, void* out, const IertBatchView* batch,
                                    const IertKvView* cache, int heads, float scale, int splits,
                                    float* scratch, int* err, cudaStream_t stream) {
   const int T = batch->n_tokens, hd = cache->head_dim;
   if (T <= 0) return IERT_OK;
-  if (cache->dtype != IERT_BF16 || hd <= 0 || (hd & 7) || hd > 64 * MAX_PAIR_ITERS || splits < 1 ||
+  if (cache->dtype != IERT_BF16 || cache->keep > 0 || hd <= 0 || (hd & 7) || hd > 64 * MAX_PAIR_ITERS || splits < 1 ||
       cache->page_tokens % KEY_BLOCK != 0 || heads <= 0 || cache->kv_heads <= 0 || heads % cache->kv_heads != 0 ||
       T > 65535)
     return IERT_BAD_ARGUMENT;

@@ -20,8 +20,8 @@
 // them; the CTA that owns the newest page rotates the new key, puts the new key and value row
 // into that page's tile in shared memory, and (one CTA per kv head) writes both to the cache.
 //
-// Visible keys: [max(0, pos + 1 - W), pos] (src/layers/attention.rs:609-613); scale from the
-// caller; softmax in fp32 (src/ops/softmax.rs:11-25).
+// Visible keys: [max(0, pos + 1 - W), pos] (src/layers/attention.rs:609-613) and the cache's kept first
+// positions, whose pages are walked in front of the window's; scale from the caller; softmax in fp32 (src/ops/softmax.rs:11-25).
 #include "common.cuh"
 #include "sm100.cuh"
 #include "tma_host.cuh"
@@ -88,12 +88,13 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-// One page's rows [0, 64) of one kv head into a padded tile; rows outside [lo, hi] are zeros.
-__device__ __forceinline__ void load_page(uint8_t* tile, const __nv_bfloat16* src, int lo, int hi) {
+// One page's rows [0, 64) of one kv head into a padded tile; rows beyond hi, and rows in front of lo that are not among
+// the first `kept` rows, are zeros.
+__device__ __forceinline__ void load_page(uint8_t* tile, const __nv_bfloat16* src, int lo, int hi, int kept) {
   constexpr int CHUNKS = HD / 8;
   for (int i = threadIdx.x; i < PAGE * CHUNKS; i += THREADS) {
     const int r = i / CHUNKS, c = i % CHUNKS;
-    const bool ok = r >= lo && r <= hi;
+    const bool ok = (r >= lo || r < kept) && r <= hi;
     cp16(tile + r * ROW_BYTES + c * 16, src + (ok ? r * HD + c * 8 : 0), ok);
   }
 }
@@ -101,9 +102,7 @@ __device__ __forceinline__ void load_page(uint8_t* tile, const __nv_bfloat16* sr
 // Pages of keys a one-token step of sequence s reads (0 for a padding sequence).
 __device__ __forceinline__ int pages_of_sequence(const IertBatchView& b, const IertKvView& c, int s) {
   if (b.slot_ids[s] < 0) return 0;
-  const int pos = b.pos0[s] + (b.cu_q[s + 1] - b.cu_q[s]) - 1;
-  const int j_min = iert_first_visible(pos, c.window, c.chunk);
-  return pos / PAGE + 1 - j_min / PAGE;
+  return iert_page_walk(c, b.pos0[s] + (b.cu_q[s + 1] - b.cu_q[s]) - 1, PAGE).n;
 }
 
 // Into how many parts a sequence of `my_pages` pages is cut when the sequences of the step have
@@ -166,19 +165,19 @@ attention_decode_tc_kernel(DecodeTcParams p, IertBatchView b, IertKvView c) {
     return;
   }
   const int pos = b.pos0[s] + (t - b.cu_q[s]);
-  const int j_min = iert_first_visible(pos, c.window, c.chunk);
-  const int pg_lo = j_min / PAGE, pg_hi = pos / PAGE + 1;           // logical pages [pg_lo, pg_hi)
+  const IertPageWalk walk = iert_page_walk(c, pos, PAGE);
+  const int j_min = walk.j_min;
   int n_splits = p.splits;
   if (p.target_ctas > 0 && p.splits > 1) {
     __shared__ int red[WARPS];
-    n_splits = balanced_parts(b, c, pg_hi - pg_lo, p.splits, p.target_ctas, gridDim.x, red);
+    n_splits = balanced_parts(b, c, walk.n, p.splits, p.target_ctas, gridDim.x, red);
     if (split >= n_splits) return;                     // this sequence is cut into fewer parts
   }
-  const int per = (pg_hi - pg_lo + n_splits - 1) / n_splits;
-  const int my_lo = pg_lo + split * per, my_hi = min(pg_hi, my_lo + per);
+  const int per = (walk.n + n_splits - 1) / n_splits;
+  const int my_lo = split * per, my_hi = min(walk.n, my_lo + per);      // this CTA's part of the walk
 
   // this CTA's range holds the newest page and the kernel has to supply the newest row itself
-  const bool own_new_row = p.rope && p.store && my_lo < my_hi && my_hi == pg_hi;
+  const bool own_new_row = p.rope && p.store && my_lo < my_hi && my_hi == walk.n;
   const int half = p.rotary_dim / 2;
   if (p.rope) {                                          // angles: no dependency on the kernel before
     for (int k = threadIdx.x; k < half; k += THREADS) {
@@ -188,16 +187,17 @@ attention_decode_tc_kernel(DecodeTcParams p, IertBatchView b, IertKvView c) {
       cs_tab[half + k] = sn;
     }
   }
-  auto issue = [&](int pg, int buf) {
-    const int page = c.page_table[(size_t)slot * c.table_width + pg % c.ring_pages];
+  auto issue = [&](int i, int buf) {
+    const int pg = iert_walk_page(walk, i);
+    const int page = c.page_table[(size_t)slot * c.table_width + iert_table_entry(c, pg)];
     const bool ok = page >= 0 && page < c.n_pages;
     if (!ok && threadIdx.x == 0) atomicOr(p.err, IERT_ERR_PAGE_RANGE);
     const size_t off = (((size_t)(ok ? page : 0) * c.kv_heads + kvh) * PAGE) * HD;
     const int lo = ok ? max(0, j_min - pg * PAGE) : PAGE;
     int hi = ok ? min(PAGE - 1, pos - pg * PAGE) : -1;
     if (own_new_row && pg == pos / PAGE) --hi;           // the newest row comes from the projection, below
-    load_page(k_tile(buf), (const __nv_bfloat16*)c.k + off, lo, hi);
-    load_page(v_tile(buf), (const __nv_bfloat16*)c.v + off, lo, hi);
+    load_page(k_tile(buf), (const __nv_bfloat16*)c.k + off, lo, hi, c.keep - pg * PAGE);
+    load_page(v_tile(buf), (const __nv_bfloat16*)c.v + off, lo, hi, c.keep - pg * PAGE);
   };
   // queries of the group: rows 0..n_g-1 of a 16-row tile, the other rows zero
   const __nv_bfloat16* tok_row = p.qkv + (size_t)t * ((size_t)(p.heads + 2 * c.kv_heads) * HD);
@@ -237,7 +237,7 @@ attention_decode_tc_kernel(DecodeTcParams p, IertBatchView b, IertKvView c) {
   // behind the first pages.  `early`: none of the first NSTAGE - 1
   // pages is the newest page (whose last row the kernel before this one writes), and a page of
   // a ring cannot be overwritten while it is read (the newest key lands in the newest page).
-  const bool early = my_lo + NSTAGE - 1 <= pos / PAGE;
+  const bool early = my_lo + NSTAGE - 1 < walk.n;
   if (!early) pdl_wait();
   if (!early) load_queries();
 #pragma unroll
@@ -263,7 +263,7 @@ attention_decode_tc_kernel(DecodeTcParams p, IertBatchView b, IertKvView c) {
     }
     __syncthreads();
     if (slice == 0) {
-      const int page = c.page_table[(size_t)slot * c.table_width + (pos / PAGE) % c.ring_pages];
+      const int page = c.page_table[(size_t)slot * c.table_width + iert_table_entry(c, pos / PAGE)];
       if (page >= 0 && page < c.n_pages) {
         const size_t off = ((((size_t)page * c.kv_heads + kvh) * PAGE) + pos % PAGE) * HD;
         for (int d = threadIdx.x; d < HD; d += THREADS) {
@@ -282,11 +282,11 @@ attention_decode_tc_kernel(DecodeTcParams p, IertBatchView b, IertKvView c) {
   for (int n = 0; n < KSTEPS * 2; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
   float m_row = -INFINITY, l_row = 0.f;          // row g (a head of the group); rows >= 8 are padding
 
-  for (int pg = my_lo; pg < my_hi; ++pg) {
-    const int buf = (pg - my_lo) % NSTAGE;
-    if (pg + NSTAGE - 1 < my_hi) issue(pg + NSTAGE - 1, (pg - my_lo + NSTAGE - 1) % NSTAGE);
+  for (int at = my_lo; at < my_hi; ++at) {
+    const int pg = iert_walk_page(walk, at), buf = (at - my_lo) % NSTAGE;
+    if (at + NSTAGE - 1 < my_hi) issue(at + NSTAGE - 1, (at - my_lo + NSTAGE - 1) % NSTAGE);
     cp_commit();
-    if (early && pg == my_lo) cp_wait<1>();      // the queries' group is the second youngest here
+    if (early && at == my_lo) cp_wait<1>();      // the queries' group is the second youngest here
     else cp_wait<NSTAGE - 1>();
     __syncthreads();
     if (own_new_row && pg == pos / PAGE) {               // the newest row of the newest page
@@ -297,7 +297,7 @@ attention_decode_tc_kernel(DecodeTcParams p, IertBatchView b, IertKvView c) {
       }
       __syncthreads();
     }
-    if (pg == my_lo) {
+    if (at == my_lo) {
 #pragma unroll
       for (int ks = 0; ks < KSTEPS; ++ks)
         ldsm4(qf[ks], q_tile + (lane & 15) * ROW_BYTES + (ks * 16 + (lane >> 4) * 8) * 2);
@@ -320,7 +320,7 @@ attention_decode_tc_kernel(DecodeTcParams p, IertBatchView b, IertKvView c) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int j = jbase + n * 8 + tq * 2 + e;
-        v[n][e] = (j >= j_min && j <= pos) ? (CAP ? softcap_l2(sc[n][e], p.cap_k2, p.cap_l2e) : sc[n][e] * p.scale_log2e) : -INFINITY;
+        v[n][e] = ((j >= j_min || j < c.keep) && j <= pos) ? (CAP ? softcap_l2(sc[n][e], p.cap_k2, p.cap_l2e) : sc[n][e] * p.scale_log2e) : -INFINITY;
         mx = fmaxf(mx, v[n][e]);
       }
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -464,17 +464,17 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     return;
   }
   const int pos = b.pos0[s] + (t - b.cu_q[s]);
-  const int j_min = iert_first_visible(pos, c.window, c.chunk);
-  const int pg_lo = j_min / PAGE, pg_hi = pos / PAGE + 1;
+  const IertPageWalk walk = iert_page_walk(c, pos, PAGE);
+  const int j_min = walk.j_min;
   int n_splits = p.splits;
   if (p.target_ctas > 0 && p.splits > 1) {
-    n_splits = balanced_parts(b, c, pg_hi - pg_lo, p.splits, p.target_ctas, gridDim.x, red);
+    n_splits = balanced_parts(b, c, walk.n, p.splits, p.target_ctas, gridDim.x, red);
     if (split >= n_splits) return;
   }
-  const int per = (pg_hi - pg_lo + n_splits - 1) / n_splits;
-  const int my_lo = pg_lo + split * per, my_hi = min(pg_hi, my_lo + per);
+  const int per = (walk.n + n_splits - 1) / n_splits;
+  const int my_lo = split * per, my_hi = min(walk.n, my_lo + per);      // this CTA's part of the walk
   const bool fused = p.rope && p.store;
-  const bool own_new_row = fused && my_lo < my_hi && my_hi == pg_hi;
+  const bool own_new_row = fused && my_lo < my_hi && my_hi == walk.n;
   const int half = p.rotary_dim / 2;
 
   if (threadIdx.x == 0) {
@@ -494,16 +494,16 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     for (int base = my_lo; base < my_hi; base += 32) {
       const int mine = base + lane;
       int page = -1;
-      if (mine < my_hi) page = c.page_table[(size_t)slot * c.table_width + mine % c.ring_pages];
+      if (mine < my_hi) page = c.page_table[(size_t)slot * c.table_width + iert_table_entry(c, iert_walk_page(walk, mine))];
       for (int k = 0; k < 32 && base + k < my_hi; ++k) {
-        const int pg = base + k, i = pg - my_lo, buf = i % NSTAGE;
+        const int i = base + k - my_lo, buf = i % NSTAGE;
         const int pgid = __shfl_sync(0xffffffffu, page, k);
         const bool ok = pgid >= 0 && pgid < c.n_pages;
         if (lane != 0 || stop) continue;
         if (abort_s) { stop = true; continue; }
         if (!ok) atomicOr(p.err, IERT_ERR_PAGE_RANGE);
         // without the fused cache write the kernel in front wrote the newest row: wait for it first
-        if (!fused && !waited && pg == pos / PAGE) { pdl_wait(); waited = true; }
+        if (!fused && !waited && base + k == walk.n - 1) { pdl_wait(); waited = true; }
         if (i >= NSTAGE && !wait_or_abort(&empty_bar[buf], ((i / NSTAGE) - 1) & 1, &abort_s)) {
           // the slot may still be in use: nothing more is asked for
           if (!abort_s) atomicOr(p.err, IERT_ERR_WAIT_EXPIRED);
@@ -579,7 +579,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   }
   consumer_sync();
   if (own_new_row && slice == 0) {
-    const int page = c.page_table[(size_t)slot * c.table_width + (pos / PAGE) % c.ring_pages];
+    const int page = c.page_table[(size_t)slot * c.table_width + iert_table_entry(c, pos / PAGE)];
     if (page >= 0 && page < c.n_pages) {
       const size_t off = ((((size_t)page * c.kv_heads + kvh) * PAGE) + pos % PAGE) * HD;
       for (int d = threadIdx.x; d < HD; d += THREADS) {
@@ -599,8 +599,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   for (int n = 0; n < KSTEPS * 2; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
   float m_row = -INFINITY, l_row = 0.f;
 
-  for (int pg = my_lo; pg < my_hi; ++pg) {
-    const int i = pg - my_lo, buf = i % NSTAGE;
+  for (int at = my_lo; at < my_hi; ++at) {
+    const int i = at - my_lo, pg = iert_walk_page(walk, at), buf = i % NSTAGE;
     if (!wait_or_abort(&full_bar[buf], (i / NSTAGE) & 1, &abort_s)) {
       if (lane == 0 && !abort_s) atomicOr(p.err, IERT_ERR_WAIT_EXPIRED);
       __syncwarp();
@@ -608,7 +608,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       break;
     }
     // this warp's 16 positions of the page: rows [16 warp, 16 warp + 16)
-    const int row_lo = max(0, j_min - pg * PAGE);
+    const int row_lo = max(0, j_min - pg * PAGE), row_keep = c.keep - pg * PAGE;
     int row_hi = min(PAGE - 1, pos - pg * PAGE);
     const bool patch = own_new_row && pg == pos / PAGE;
     if (patch) --row_hi;                                      // the newest row comes from the projection
@@ -616,7 +616,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     bool wrote = false;
     if (row_lo > w0 || row_hi < w0 + 15) {                    // rows of the values that must not count
       for (int r = w0; r < w0 + 16; ++r) {
-        if ((r >= row_lo && r <= row_hi) || (patch && r == pos % PAGE)) continue;      // (the patched row: below)
+        if (((r >= row_lo || r < row_keep) && r <= row_hi) || (patch && r == pos % PAGE)) continue;      // (the patched row: below)
 #pragma unroll
         for (int bx = 0; bx < BOXES; ++bx)
           reinterpret_cast<uint32_t*>(v_tile(buf) + bx * BOX_BYTES + r * 128)[lane] = 0u;
@@ -648,7 +648,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int j = jbase + n * 8 + tq * 2 + e;
-        v[n][e] = (j >= j_min && j <= pos) ? (CAP ? softcap_l2(sc[n][e], p.cap_k2, p.cap_l2e) : sc[n][e] * p.scale_log2e) : -INFINITY;
+        v[n][e] = ((j >= j_min || j < c.keep) && j <= pos) ? (CAP ? softcap_l2(sc[n][e], p.cap_k2, p.cap_l2e) : sc[n][e] * p.scale_log2e) : -INFINITY;
         mx = fmaxf(mx, v[n][e]);
       }
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -748,9 +748,8 @@ __global__ void attention_decode_tc_combine_kernel(DecodeTcParams p, IertBatchVi
   const bool live = s_ >= 0 && b.slot_ids[s_] >= 0;
   if (p.target_ctas > 0 && p.splits > 1 && live) {
     const int pos = b.pos0[s_] + (t - b.cu_q[s_]);
-    const int j_min = iert_first_visible(pos, c.window, c.chunk);
     const int group = p.heads / c.kv_heads;
-    n_splits = balanced_parts(b, c, pos / PAGE + 1 - j_min / PAGE, p.splits, p.target_ctas,
+    n_splits = balanced_parts(b, c, iert_page_walk(c, pos, PAGE).n, p.splits, p.target_ctas,
                               c.kv_heads * ((group + p.gt - 1) / p.gt), red);
   }
   pdl_wait();                  // everything below may depend on the kernel before

@@ -4,7 +4,8 @@
 // running maximum and sum, so the memory it needs does not grow with the context.
 //
 //   scores  s_j = (q . k_j) * scale for j in [j_min, pos], causal by construction
-//   window  j_min = pos - (W - 1) (the last W keys, the current one included); chunk: j_min = pos - pos % C
+//   window  j_min = pos - (W - 1) (the last W keys, the current one included); chunk: j_min = pos - pos % C;
+//           keep: positions [0, keep) are visible besides
 //   weights softmax over the visible keys; output = sum_j p_j v_j
 //   softcap c > 0: s_j <- c tanh(s_j / c) before the softmax
 //   sink    (optional, fp32 per head): one more term exp(sink[head]) in the denominator, with no value
@@ -47,6 +48,9 @@ attention_plain_kernel(const T* __restrict__ qkv, T* __restrict__ out, IertBatch
   const int pos0 = b.pos0[s];
   const int pos = pos0 + (t - q_begin);
   const int j_min = iert_first_visible(pos, c.window, c.chunk);
+  const int n_keep = min(c.keep, j_min);           // kept first positions in front of the window
+  const int n_keys = n_keep + pos - j_min + 1;     // visible keys, numbered i: the kept ones, then [j_min, pos]
+  auto key_of = [&](int i) { return i < n_keep ? i : j_min + i - n_keep; };
   const int kvh = head / (heads / nkv);
 
   const T* q = qkv + (size_t)t * row_elems + (size_t)head * hd;
@@ -58,8 +62,8 @@ attention_plain_kernel(const T* __restrict__ qkv, T* __restrict__ out, IertBatch
 #pragma unroll
   for (int i = 0; i < MAX_DIMS_PER_THREAD; ++i) acc[i] = 0.f;
 
-  for (int j0 = j_min; j0 <= pos; j0 += THREADS) {
-    const int j = j0 + threadIdx.x;
+  for (int i0 = 0; i0 < n_keys; i0 += THREADS) {
+    const int j = key_of(i0 + threadIdx.x);
     float sc = -INFINITY;
     if (j <= pos) {
       const T* k;
@@ -84,7 +88,7 @@ attention_plain_kernel(const T* __restrict__ qkv, T* __restrict__ out, IertBatch
     m = m_new;
     p_s[threadIdx.x] = p;
     __syncthreads();
-    const int n_in_chunk = min(THREADS, pos - j0 + 1);
+    const int n_in_chunk = min(THREADS, n_keys - i0);
 #pragma unroll
     for (int i = 0; i < MAX_DIMS_PER_THREAD; ++i) {
       const int d = threadIdx.x + i * THREADS;
@@ -95,11 +99,11 @@ attention_plain_kernel(const T* __restrict__ qkv, T* __restrict__ out, IertBatch
         if (pj == 0.f) continue;
         const T* v;
         if (PAGED) {
-          const long long off = kv_row_offset(c, slot, j0 + jj, kvh, nullptr);
+          const long long off = kv_row_offset(c, slot, key_of(i0 + jj), kvh, nullptr);
           if (off < 0) continue;
           v = (const T*)c.v + off;
         } else {
-          v = qkv + (size_t)(q_begin + (j0 + jj - pos0)) * row_elems + (size_t)(heads + nkv + kvh) * hd;
+          v = qkv + (size_t)(q_begin + (key_of(i0 + jj) - pos0)) * row_elems + (size_t)(heads + nkv + kvh) * hd;
         }
         a = fmaf(pj, to_f32(v[d]), a);
       }

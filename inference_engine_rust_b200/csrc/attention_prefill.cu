@@ -9,7 +9,8 @@
 //   to is in the step) through cp.async into double-buffered shared memory whose rows are
 //   padded by 16 bytes, which makes every ldmatrix conflict-free for any head size.
 //   Visible keys of query i: j in [max(0, i - (W - 1)), i] (src/layers/attention.rs:364-368);
-//   tiles entirely outside are never loaded, tiles entirely inside skip the mask.
+//   tiles entirely outside are never loaded, tiles entirely inside skip the mask.  `keep` first positions of the
+//   sequence stay visible: their tiles are visited in front of the window's.
 //
 // Formulas: src/layers/attention.rs:357-415, src/ops/softmax.rs:11-25.
 #include "common.cuh"
@@ -79,7 +80,7 @@ __device__ __forceinline__ void load_tile(uint8_t* tile, const __nv_bfloat16* sr
 
 __global__ void __launch_bounds__(THREADS)
 attention_prefill_kernel(const __nv_bfloat16* __restrict__ qkv, __nv_bfloat16* __restrict__ out,
-                         IertBatchView b, int heads, int kv_heads, int window, int chunk, float scale_log2e,
+                         IertBatchView b, int heads, int kv_heads, int window, int chunk, int keep, float scale_log2e,
                          const float* __restrict__ sink, float cap_k2, float cap_l2e) {
   extern __shared__ __align__(16) uint8_t smem[];
   uint8_t* q_tile = smem;
@@ -102,11 +103,14 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ qkv, __nv_bfloat16* _
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
   const int i_hi = min(len, i0 + BM) - 1;               // last valid query of the tile
   const int j_lo = iert_first_visible(i0, window, chunk);
-  const int kt_lo = j_lo / BN, kt_hi = i_hi / BN;       // key tiles to visit, inclusive
+  const int kt_lo = j_lo / BN, kt_hi = i_hi / BN;       // key tiles of the window, inclusive
+  const int n_kept = iert_kept_blocks(keep, BN, kt_lo); // tiles of kept first positions in front of them
+  const int n_tiles = n_kept + kt_hi - kt_lo + 1;
+  auto tile_at = [&](int it) { return it < n_kept ? it : kt_lo + it - n_kept; };
 
   load_tile<BM>(q_tile, q_src, ld, len - i0);
-  load_tile<BN>(k_tile(0), k_src + (long long)kt_lo * BN * ld, ld, len - kt_lo * BN);
-  load_tile<BN>(v_tile(0), v_src + (long long)kt_lo * BN * ld, ld, len - kt_lo * BN);
+  load_tile<BN>(k_tile(0), k_src + (long long)tile_at(0) * BN * ld, ld, len - tile_at(0) * BN);
+  load_tile<BN>(v_tile(0), v_src + (long long)tile_at(0) * BN * ld, ld, len - tile_at(0) * BN);
   cp_async_commit();
 
   uint32_t q_frag[Q_IN_REGS ? KSTEPS : 1][4];
@@ -116,11 +120,12 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ qkv, __nv_bfloat16* _
   float m_row[2] = {-INFINITY, -INFINITY}, l_row[2] = {0.f, 0.f};   // rows g and g + 8 of the warp's 16
   const int qi[2] = {i0 + warp * 16 + g, i0 + warp * 16 + g + 8};   // their positions in the sequence
 
-  for (int kt = kt_lo; kt <= kt_hi; ++kt) {
-    const int buf = (kt - kt_lo) & 1;
-    if (kt < kt_hi) {                                   // prefetch the next tile into the other buffer
-      load_tile<BN>(k_tile(buf ^ 1), k_src + (long long)(kt + 1) * BN * ld, ld, len - (kt + 1) * BN);
-      load_tile<BN>(v_tile(buf ^ 1), v_src + (long long)(kt + 1) * BN * ld, ld, len - (kt + 1) * BN);
+  for (int it = 0; it < n_tiles; ++it) {
+    const int buf = it & 1, kt = tile_at(it);
+    if (it + 1 < n_tiles) {                             // prefetch the next tile into the other buffer
+      const int nt = tile_at(it + 1);
+      load_tile<BN>(k_tile(buf ^ 1), k_src + (long long)nt * BN * ld, ld, len - nt * BN);
+      load_tile<BN>(v_tile(buf ^ 1), v_src + (long long)nt * BN * ld, ld, len - nt * BN);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -128,7 +133,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ qkv, __nv_bfloat16* _
     }
     __syncthreads();
     if constexpr (Q_IN_REGS) {
-      if (kt == kt_lo) {
+      if (it == 0) {
 #pragma unroll
         for (int ks = 0; ks < KSTEPS; ++ks)
           ldmatrix_x4(q_frag[ks], q_tile + (warp * 16 + (lane & 15)) * ROW_BYTES + (ks * 16 + (lane >> 4) * 8) * 2);
@@ -166,7 +171,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ qkv, __nv_bfloat16* _
         float v = cap_l2e > 0.f ? softcap_l2(sc[n][e], cap_k2, cap_l2e) : sc[n][e] * scale_log2e;
         if (need_mask) {
           const int j = j0 + n * 8 + tq * 2 + (e & 1), i = qi[e >> 1];
-          const bool vis = j <= i && j < len && j >= iert_first_visible(i, window, chunk);
+          const bool vis = j <= i && j < len && (j >= iert_first_visible(i, window, chunk) || j < keep);
           if (!vis) v = -INFINITY;
         }
         sc[n][e] = v;
@@ -242,7 +247,7 @@ IERT_API int iert_attention_prefill_head_dim() { return HD; }
 // out: bf16 [T, heads * HEAD_DIM].  Every sequence of the step starts at position 0.
 // max_q_len: the longest sequence of the step (sizes the grid).
 IERT_API int iert_attention_prefill(const void* qkv, void* out, const IertBatchView* batch, int heads,
-                                    int kv_heads, int window, int chunk, float scale, int max_q_len, const float* sink,
+                                    int kv_heads, int window, int chunk, int keep, float scale, int max_q_len, const float* sink,
                                     float softcap, cudaStream_t stream) {
   if (batch->n_tokens <= 0 || max_q_len <= 0) return IERT_OK;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || heads > 65535 || batch->n_seqs > 65535)
@@ -258,7 +263,7 @@ IERT_API int iert_attention_prefill(const void* qkv, void* out, const IertBatchV
   }
   dim3 grid((max_q_len + BM - 1) / BM, heads, batch->n_seqs);
   attention_prefill_kernel<<<grid, THREADS, smem, stream>>>(
-      (const __nv_bfloat16*)qkv, (__nv_bfloat16*)out, *batch, heads, kv_heads, window, chunk,
+      (const __nv_bfloat16*)qkv, (__nv_bfloat16*)out, *batch, heads, kv_heads, window, chunk, keep,
       scale * 1.4426950408889634f, sink, softcap > 0.f ? 2.0f * scale * 1.4426950408889634f / softcap : 0.f,
       softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
   cudaError_t e = cudaGetLastError();

@@ -26,7 +26,8 @@
 //   Every mbarrier wait is bounded; on expiry the kernel records IERT_ERR_WAIT_EXPIRED, frees
 //   its TMEM and returns.
 //
-// Visible keys of query i: j in [max(0, i - (W - 1)), i] (src/layers/attention.rs:364-368);
+// Visible keys of query i: j in [max(0, i - (W - 1)), i] (src/layers/attention.rs:364-368), and the `keep` first
+// positions of the sequence, whose tiles are visited in front of the window's;
 // formulas src/layers/attention.rs:357-415, src/ops/softmax.rs:11-25.
 #include "common.cuh"
 #include "sm100.cuh"
@@ -55,7 +56,7 @@ constexpr uint32_t O_COL = 128;
 
 struct PrefillTcParams {
   __nv_bfloat16* out;         // [T, heads * HD]
-  int heads, kv_heads, window, chunk;
+  int heads, kv_heads, window, chunk, keep;
   float scale_log2e;
   float cap_k2, cap_l2e;   // a soft cap on the scores (cap_l2e > 0): see softcap_l2
   const float* sink;       // optional [heads]: a bare logit per head that adds exp(sink) to every row's denominator only
@@ -135,7 +136,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   const int i_hi = min(len, i0 + BM) - 1;
   const int j_lo = iert_first_visible(i0, p.window, p.chunk);
   const int kt_lo = j_lo / BN, kt_hi = i_hi / BN;
-  const int n_tiles = kt_hi - kt_lo + 1;
+  const int n_kept = iert_kept_blocks(p.keep, BN, kt_lo);    // tiles of kept first positions in front of the window
+  const int n_tiles = n_kept + kt_hi - kt_lo + 1;
+  auto tile_at = [&](int it) { return it < n_kept ? it : kt_lo + it - n_kept; };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
   if (threadIdx.x == 0) {
@@ -171,7 +174,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         mbar_expect_tx(&k_full[st], NSUB * KV_SUB_BYTES);
         for (int sb = 0; sb < NSUB; ++sb)
           tma_load_2d(k_s + (st * NSUB + sb) * KV_SUB_BYTES, &map_kv, &k_full[st], k_col + 64 * sb,
-                      q_begin + (kt_lo + it) * BN);
+                      q_begin + tile_at(it) * BN);
         return true;
       };
       auto load_v = [&](int it) -> bool {
@@ -180,7 +183,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         mbar_expect_tx(&v_full[st], NSUB * KV_SUB_BYTES);
         for (int sb = 0; sb < NSUB; ++sb)
           tma_load_2d(v_s + (st * NSUB + sb) * KV_SUB_BYTES, &map_kv, &v_full[st], v_col + 64 * sb,
-                      q_begin + (kt_lo + it) * BN);
+                      q_begin + tile_at(it) * BN);
         return true;
       };
       ok = load_k(0);
@@ -239,7 +242,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const uint32_t lane_bits = (uint32_t)(warp * 32) << 16;
     float m_used = -INFINITY, l = 0.f;
     for (int it = 0; ok && it < n_tiles; ++it) {
-      const int st = it & 1, j0 = (kt_lo + it) * BN;
+      const int st = it & 1, j0 = tile_at(it) * BN;
       if (!wait_bar(&s_full[st], (it >> 1) & 1, abort_flag)) { ok = false; break; }
       tc_fence_after();
       float sc[BN];
@@ -264,7 +267,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
         for (int c = 0; c < BN; ++c) {
           const int j = j0 + c;
-          const bool vis = j <= i && j < len && j >= i_lo;
+          const bool vis = j <= i && j < len && (j >= i_lo || j < p.keep);
           if (!vis) sc[c] = -INFINITY;
         }
       }
@@ -370,7 +373,7 @@ IERT_API int iert_attention_prefill_tc_available() { return 1; }
 // Same contract as iert_attention_prefill; additionally qkv must be 16-byte aligned.  Returns
 // IERT_BAD_ARGUMENT (nothing launched) when the tensor map cannot be made.
 IERT_API int iert_attention_prefill_tc(const void* qkv, void* out, const IertBatchView* batch, int heads,
-                                       int kv_heads, int window, int chunk, float scale, int max_q_len, int* err,
+                                       int kv_heads, int window, int chunk, int keep, float scale, int max_q_len, int* err,
                                        const float* sink, float softcap, cudaStream_t stream) {
   if (batch->n_tokens <= 0 || max_q_len <= 0) return IERT_OK;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || (max_q_len + BM - 1) / BM > 65535 || batch->n_seqs > 65535 ||
@@ -383,7 +386,7 @@ IERT_API int iert_attention_prefill_tc(const void* qkv, void* out, const IertBat
     return IERT_BAD_ARGUMENT;
   PrefillTcParams p;
   p.out = (__nv_bfloat16*)out;
-  p.heads = heads; p.kv_heads = kv_heads; p.window = window; p.chunk = chunk;
+  p.heads = heads; p.kv_heads = kv_heads; p.window = window; p.chunk = chunk; p.keep = keep;
   p.scale_log2e = scale * 1.4426950408889634f;
   p.sink = sink;
   p.cap_k2 = softcap > 0.f ? 2.0f * scale * 1.4426950408889634f / softcap : 0.f;
@@ -406,7 +409,7 @@ IERT_API int iert_attention_prefill_tc(const void* qkv, void* out, const IertBat
 #else   // other head sizes: the mma.sync kernel serves them
 
 IERT_API int iert_attention_prefill_tc_available() { return 0; }
-IERT_API int iert_attention_prefill_tc(const void*, void*, const IertBatchView*, int, int, int, int, float, int, int*, const float*,
+IERT_API int iert_attention_prefill_tc(const void*, void*, const IertBatchView*, int, int, int, int, int, float, int, int*, const float*,
                                        float, cudaStream_t) {
   return IERT_BAD_ARGUMENT;
 }

@@ -35,7 +35,7 @@ class KvView(Structure):
     _fields_ = [("k", c_void_p), ("v", c_void_p), ("page_table", c_void_p),
                 ("table_width", c_int), ("ring_pages", c_int), ("page_tokens", c_int),
                 ("n_pages", c_int), ("kv_heads", c_int), ("head_dim", c_int),
-                ("dtype", c_int), ("window", c_int), ("chunk", c_int)]
+                ("dtype", c_int), ("window", c_int), ("chunk", c_int), ("keep", c_int), ("keep_pages", c_int)]
 
 
 class BatchView(Structure):
@@ -116,7 +116,7 @@ def _declare(lib) -> None:
     sigs = {
         "iert_embed_gather": [P, c_int, P, P, c_int, c_int, c_int, c_float, P, POINTER(NormAhead), S],
         "iert_rmsnorm": [P, P, c_int, P, c_int, P, c_int, c_int, c_float, S],
-        "iert_rope_kv_store": [P, c_int, POINTER(BatchView), POINTER(KvView), P, c_int, c_int, c_int, c_int, P, S],
+        "iert_rope_kv_store": [P, c_int, POINTER(BatchView), POINTER(KvView), P, c_int, c_int, c_float, c_int, c_int, P, S],
         "iert_silu_mul": [P, P, c_int, c_int, c_int, S],
         "iert_gated_act_mul": [P, P, c_int, c_int, c_int, POINTER(GatedAct), S],
         "iert_add_into": [P, P, c_int, c_longlong, S],
@@ -142,8 +142,10 @@ def _declare(lib) -> None:
         "iert_latent_attention_prompt": [P, LL, P, c_int, POINTER(BatchView), c_int, c_int, c_int, c_float, P, S],
         "iert_latent_attention_decode": [P, LL, P, P, P, c_int, POINTER(BatchView), POINTER(KvView), c_int, c_int, c_int, c_int,
                                          c_float, P, P, P, S],
-        "iert_latent_prep": [P, LL, c_int, c_int, c_int, c_int, P, c_float, P, c_int, c_int, c_float, P, P, LL, c_int, P, c_int,
-                             POINTER(BatchView), POINTER(KvView), c_int, P, S],
+        "iert_latent_prep": [P, LL, P, LL, P, LL, P, LL, c_int, c_int, c_int, c_int, c_int, P, P, c_float, P, c_float, c_int,
+                             c_float, P, P, LL, c_int, P, P, c_int, POINTER(BatchView), POINTER(KvView), c_int, P, S],
+        "iert_layernorm": [P, P, c_int, c_int, c_float, P, P, P, P, P, P, c_int, S],
+        "iert_embed_pairs": [P, c_int, P, c_int, P, P, c_int, c_int, c_int, c_float, c_int, LL, LL, P, LL, POINTER(BatchView), P, S],
         "iert_head_gate_mul": [P, c_int, P, c_int, c_int, P, c_int, POINTER(BatchView), S],
         "iert_token_shift": [P, c_int, LL, P, LL, LL, P, c_int, c_int, P, POINTER(BatchView), S],
         "iert_wkv_decay": [P, LL, c_int, P, P, c_int, P, P, c_int, LL, c_int, P, LL, LL, POINTER(BatchView), S],
@@ -153,9 +155,9 @@ def _declare(lib) -> None:
         "iert_moe_scale": [P, c_int, LL, P, c_int, c_int, c_int, P, P, LL, P, c_int, S],
         "iert_router_grouped": [P, LL, LL, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
                                 P, P, P, P, S],
-        "iert_qkv_prep": [P, LL, P, P, c_int, POINTER(BatchView), POINTER(KvView), c_int, c_int, c_int, P, c_int, c_int, P, P,
-                          c_float, c_int, P, S],
-        "iert_gate_mul": [P, P, LL, P, c_int, c_int, c_int, c_int, c_int, S],
+        "iert_qkv_prep": [P, LL, P, P, c_int, POINTER(BatchView), POINTER(KvView), c_int, c_int, c_int, P, c_int, c_float, c_int,
+                          P, P, c_float, P, LL, c_float, c_int, P, S],
+        "iert_gate_mul": [P, P, LL, c_int, P, c_int, c_int, c_int, c_int, c_int, S],
         "iert_add_normed": [P, P, P, P, c_int, c_int, c_int, c_float, S],
         "iert_cast_rows": [P, P, P, c_int, LL, S],
         "iert_scale_values": [P, LL, c_float, S],
@@ -259,9 +261,9 @@ def sm_count() -> int:
 
 
 def rope_kv_store(qkv, batch: BatchView, kv: KvView, inv_freq, heads: int, rotary_dim: int,
-                  pairing: int, write_cache: bool, err, stream) -> None:
+                  pairing: int, write_cache: bool, err, stream, rot_mul: float = 1.0) -> None:
     check(core().iert_rope_kv_store(qkv.data_ptr(), dtype_code(qkv.dtype), byref(batch), byref(kv),
-                                    inv_freq.data_ptr(), heads, rotary_dim, pairing,
+                                    inv_freq.data_ptr(), heads, rotary_dim, rot_mul, pairing,
                                     1 if write_cache else 0, err.data_ptr(), stream), "rope_kv_store")
 
 
@@ -281,11 +283,11 @@ def kv_store(qkv, batch: BatchView, kv: KvView, heads: int, err, stream) -> None
 
 
 def rotate_qk(qkv, batch: BatchView, inv_freq, heads: int, kv_heads: int, head_dim: int, rotary_dim: int,
-              pairing: int, err, stream) -> None:
-    """Rotate the step's queries and keys in place; nothing is stored."""
+              pairing: int, err, stream, rot_mul: float = 1.0) -> None:
+    """Rotate the step's queries and keys in place (cosine and sine times `rot_mul`); nothing is stored."""
     geometry = KvView(k=None, v=None, page_table=None, table_width=0, ring_pages=1, page_tokens=1, n_pages=0,
                       kv_heads=kv_heads, head_dim=head_dim, dtype=dtype_code(qkv.dtype), window=0)
-    rope_kv_store(qkv, batch, geometry, inv_freq, heads, rotary_dim, pairing, False, err, stream)
+    rope_kv_store(qkv, batch, geometry, inv_freq, heads, rotary_dim, pairing, False, err, stream, rot_mul)
 
 
 def silu_mul(gu, out, n_tokens: int, inter: int, stream) -> None:
@@ -470,7 +472,7 @@ def _attention_lib(head_dim: int):
     lib = _attn_libs.get(head_dim)
     if lib is None:
         lib = build.load_library(*build.attention_library(head_dim))
-        lib.iert_attention_prefill.argtypes = [c_void_p, c_void_p, POINTER(BatchView), c_int, c_int, c_int, c_int,
+        lib.iert_attention_prefill.argtypes = [c_void_p, c_void_p, POINTER(BatchView), c_int, c_int, c_int, c_int, c_int,
                                                c_float, c_int, c_void_p, c_float, c_void_p]
         lib.iert_attention_prefill.restype = c_int
         lib.iert_attention_decode_tc.argtypes = [c_void_p, c_void_p, POINTER(BatchView), POINTER(KvView), c_int,
@@ -480,7 +482,7 @@ def _attention_lib(head_dim: int):
                                                       c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                                                       c_void_p, c_void_p]
         lib.iert_attention_decode_tc_rope.restype = c_int
-        lib.iert_attention_prefill_tc.argtypes = [c_void_p, c_void_p, POINTER(BatchView), c_int, c_int, c_int, c_int,
+        lib.iert_attention_prefill_tc.argtypes = [c_void_p, c_void_p, POINTER(BatchView), c_int, c_int, c_int, c_int, c_int,
                                                   c_float, c_int, c_void_p, c_void_p, c_float, c_void_p]
         lib.iert_attention_prefill_tc.restype = c_int
         lib.iert_attention_prefill_tc_available.restype = c_int
@@ -493,10 +495,10 @@ def _attention_lib(head_dim: int):
 
 def attention_prefill(qkv, out, batch: BatchView, heads: int, kv_heads: int, head_dim: int, window: int,
                       scale: float, max_q_len: int, stream, err=None, legacy: bool = False, sink=None,
-                      softcap: float = 0.0, chunk: int = 0) -> bool:
+                      softcap: float = 0.0, chunk: int = 0, keep: int = 0) -> bool:
     """Flash prompt attention (bf16) over the step's own keys and values (`window` W > 0: the last W keys; `chunk`
-    C > 0: the keys of the query's own chunk of C positions).  Head sizes 64 and
-    128 run on tcgen05 with the scores and the output in tensor memory (unless `legacy`); other
+    C > 0: the keys of the query's own chunk of C positions; `keep`: the first positions of the sequence stay visible
+    whatever the two say).  Head sizes 64, 128, 192 and 256 run on tcgen05 with the scores and the output in tensor memory (unless `legacy`); other
     multiples of 16 up to 256 run the mma.sync kernel.  The library is compiled per head size
     the first time it is needed; anything else returns False and nothing is launched.  `sink` (fp32
     [heads], optional): a bare logit per head that adds exp(sink) to each row's softmax denominator only;
@@ -508,7 +510,7 @@ def attention_prefill(qkv, out, batch: BatchView, heads: int, kv_heads: int, hea
     if not legacy and err is not None and lib.iert_attention_prefill_tc_available() \
             and os.environ.get("IERT_ATTN_TC", "1") != "0":
         status = lib.iert_attention_prefill_tc(qkv.data_ptr(), out.data_ptr(), byref(batch), heads, kv_heads,
-                                               window, chunk, scale, max_q_len, err.data_ptr(),
+                                               window, chunk, keep, scale, max_q_len, err.data_ptr(),
                                                sink.data_ptr() if sink is not None else None, softcap, stream)
         if status == 0:
             launch_count += 1
@@ -516,7 +518,7 @@ def attention_prefill(qkv, out, batch: BatchView, heads: int, kv_heads: int, hea
         if status != 1:
             raise KernelError("attention_prefill_tc: the launch failed")
     status = lib.iert_attention_prefill(qkv.data_ptr(), out.data_ptr(), byref(batch), heads, kv_heads,
-                                        window, chunk, scale, max_q_len, sink.data_ptr() if sink is not None else None, softcap,
+                                        window, chunk, keep, scale, max_q_len, sink.data_ptr() if sink is not None else None, softcap,
                                         stream)
     if status == 1:
         return False
@@ -744,16 +746,22 @@ def latent_attention_decode(q, w_uk, w_uv, out, batch: BatchView, kv: KvView, H:
                                               _ptr(gate), err.data_ptr(), stream), "latent_attention_decode")
 
 
-def latent_prep(x, H: int, D: int, R: int, rank: int, wkv, eps: float, inv_freq, pairing: int, out_scale: float, c_ext, q_out,
-                q_head: int, gate_out, batch: BatchView, kv: KvView, store: bool, err, stream) -> None:
-    """From the fp32 projection rows x = [q: H x (D | R) | latent: rank | rotated key part: R | gate logits: H (if
-    `gate_out`)] to the normed latent and rotated key part `c_ext` [T, rank + R] (also the cache row, with `store`), the
-    queries `q_out` [T, H, q_head] (rotated part turned, zeros beyond D + R) and `gate_out` = sigmoid(logit) * out_scale."""
-    check(core().iert_latent_prep(x.data_ptr(), x.stride(0), H, D, R, rank, wkv.data_ptr(), eps, _ptr(inv_freq), pairing,
-                                  1 if gate_out is not None else 0, out_scale, c_ext.data_ptr(), q_out.data_ptr(), q_out.stride(0),
-                                  q_head,
-                                  _ptr(gate_out), dtype_code(c_ext.dtype), byref(batch), byref(kv), 1 if store else 0,
-                                  err.data_ptr(), stream), "latent_prep")
+def latent_prep(H: int, D: int, R: int, rank: int, eps: float, inv_freq, pairing: int, batch: BatchView, kv: KvView, err, stream, *,
+                q=None, q_out=None, q_head: int = 0, down=None, wkv=None, c_ext=None, store: bool = False, dq=None, wq=None,
+                cq=None, glog=None, gate_out=None, out_scale: float = 1.0, rot_mul: float = 1.0) -> None:
+    """The rows of latent attention with a rotated part from fp32 projections (views whose rows may be strided), each piece
+    there or not: `q` [T, H x (D | R)] -> `q_out` [T, H, q_head] (rotated part turned, zeros beyond D + R); `down`
+    [T, rank | R] -> `c_ext` [T, rank + R] (normed latent, rotated key part; also the cache row, with `store`); `dq` -> `cq`
+    (normed query latent); `glog` [T, H] -> `gate_out` = sigmoid(logit) * out_scale."""
+    some = next(t for t in (c_ext, q_out, cq) if t is not None)
+
+    def ld(t):
+        return t.stride(0) if t is not None else 0
+    check(core().iert_latent_prep(_ptr(q), ld(q), _ptr(down), ld(down), _ptr(dq), ld(dq), _ptr(glog), ld(glog), H, D, R, rank,
+                                  cq.shape[-1] if cq is not None else 0, _ptr(wkv), _ptr(wq), eps, _ptr(inv_freq), rot_mul,
+                                  pairing, out_scale, _ptr(c_ext), _ptr(q_out), ld(q_out), q_head, _ptr(cq), _ptr(gate_out),
+                                  dtype_code(some.dtype), byref(batch), byref(kv), 1 if store else 0, err.data_ptr(), stream),
+          "latent_prep")
 
 
 def head_gate_mul(attn, head: int, out, V: int, H: int, gate, batch: BatchView, stream) -> None:
@@ -771,19 +779,21 @@ def latent_decode_tc_plan(n_seqs: int, H: int, table_width: int):
 
 def latent_attention_decode_tc(q, w_uk, w_uv, out, batch: BatchView, kv: KvView, H: int, D: int, V: int, scale: float, sink,
                                hpad: int, splits: int, qa, part_m, part_l, part_acc, err, stream, rot_dim: int = 0,
-                               gate=None) -> bool:
+                               gate=None, inv_freq=None, rot_mul: float = 1.0, pairing: int = PAIR_HALF) -> bool:
     """One-token latent attention on the tensor cores (bf16, rank a multiple of 32 up to 512, pages of 64):
-    the absorbed queries, the split attention over the cached latents, the merge with the sink and W_uv.
+    the absorbed queries, the split attention over the cached latents, the merge with the sink and W_uv.  `q`: bf16 with its
+    rotated part turned already, or the fp32 projection, whose rotated part is turned here by `inv_freq`, `rot_mul`, `pairing`.
     Returns False, having launched nothing, for sizes it does not take."""
     lib = core()
     fn = lib.iert_latent_attention_decode_tc
     if not getattr(fn, "_declared", False):
-        fn.argtypes = [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, POINTER(BatchView), POINTER(KvView), c_int, c_int,
+        fn.argtypes = [c_void_p, c_int, c_longlong, c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p, POINTER(BatchView),
+                       POINTER(KvView), c_int, c_int,
                        c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_void_p]
         fn.restype = c_int
         fn._declared = True
-    status = fn(q.data_ptr(), q.stride(0), w_uk.data_ptr(), w_uv.data_ptr(), out.data_ptr(), byref(batch), byref(kv), H, D,
+    status = fn(q.data_ptr(), 1 if q.dtype == torch.float32 else 0, q.stride(0), _ptr(inv_freq), rot_mul, pairing, w_uk.data_ptr(), w_uv.data_ptr(), out.data_ptr(), byref(batch), byref(kv), H, D,
                 rot_dim, V, scale, _ptr(sink), _ptr(gate), hpad, splits, qa.data_ptr(), part_m.data_ptr(), part_l.data_ptr(), part_acc.data_ptr(),
                 err.data_ptr(), stream)
     if status == 1:
@@ -859,20 +869,39 @@ def qk_prep(proj, qkv, batch: BatchView, kv: KvView, heads: int, inv_freq, rotar
 
 
 def qkv_prep(proj, bias, qkv, batch: BatchView, kv: KvView, heads: int, dim: int, vdim: int, inv_freq, rotary_dim: int,
-             pairing: int, wq, wk, eps: float, store: bool, err, stream) -> None:
+             pairing: int, wq, wk, eps: float, store: bool, err, stream, rot_mul: float = 1.0, v_first=None, lam: float = 0.0) -> None:
     """From the fp32 projection rows that begin with [q | k | v] (+ `bias`) to the packed rows [q' | k' | v'] with every
     head padded with zeros to the cache's head size: per-head weighted RMS norm of q and k (`wq`, `wk` of length `dim`,
-    optional), rotation, one rounding, and the cache write of k' and v'."""
+    optional), rotation (cosine and sine times `rot_mul`), values mixed with another layer's (v <- (1 - lam) v + lam v_first,
+    `v_first` fp32 rows that may be strided), one rounding, and the cache write of k' and v'."""
     check(core().iert_qkv_prep(proj.data_ptr(), proj.stride(0), _ptr(bias), qkv.data_ptr(), dtype_code(qkv.dtype), byref(batch),
-                               byref(kv), heads, dim, vdim, _ptr(inv_freq), rotary_dim, pairing, _ptr(wq), _ptr(wk), eps,
+                               byref(kv), heads, dim, vdim, _ptr(inv_freq), rotary_dim, rot_mul, pairing, _ptr(wq), _ptr(wk), eps,
+                               _ptr(v_first), v_first.stride(0) if v_first is not None else 0, lam,
                                1 if store else 0, err.data_ptr(), stream), "qkv_prep")
 
 
-def gate_mul(attn, gate, out, n_tokens: int, heads: int, D: int, vdim: int, stream) -> None:
-    """out[t, h*vdim + c] = attn[t, h*D + c] * sigmoid(gate[t, h*vdim + c]); `gate` (fp32, a view whose rows may be
-    strided) may be None: the padding of the heads is dropped and nothing else."""
-    check(core().iert_gate_mul(attn.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(),
-                               dtype_code(attn.dtype), n_tokens, heads, D, vdim, stream), "gate_mul")
+def gate_mul(attn, gate, out, n_tokens: int, heads: int, D: int, vdim: int, stream, per_head: bool = False) -> None:
+    """out[t, h*vdim + c] = attn[t, h*D + c] * sigmoid(gate[t, h*vdim + c]), or with `per_head` * sigmoid(gate[t, h]);
+    `gate` (fp32, a view whose rows may be strided) may be None: the padding of the heads is dropped and nothing else."""
+    check(core().iert_gate_mul(attn.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0, 1 if per_head else 0,
+                               out.data_ptr(), dtype_code(attn.dtype), n_tokens, heads, D, vdim, stream), "gate_mul")
+
+
+def layernorm(x, out, w, b, eps: float, rows: int, stream, rows_idx=None, second=None) -> None:
+    """LayerNorm of fp32 rows with fp32 weight and bias; `second` = (w, b, out): another norm of the same rows, in the same pass."""
+    w1, b1, out1 = second if second is not None else (None, None, None)
+    check(core().iert_layernorm(x.data_ptr(), _ptr(rows_idx), rows, x.shape[-1], eps, w.data_ptr(), _ptr(b), out.data_ptr(), _ptr(w1),
+                                _ptr(b1), _ptr(out1), dtype_code(out.dtype), stream), "layernorm")
+
+
+def embed_pairs(table, pairs, ids, x, scale: float, buckets: int, mul_prev: int, mul_cur: int, last, batch: BatchView, err,
+                stream) -> None:
+    """x[t] = table[ids[t]] * scale + pairs[row], row = (id in front * mul_prev + ids[t] * mul_cur) mod buckets, or `buckets` for
+    a sequence's first token; `last` (int32 [slots, n], column 0) keeps each sequence's last token from step to step."""
+    vocab, hidden = table.shape
+    check(core().iert_embed_pairs(table.data_ptr(), dtype_code(table.dtype), pairs.data_ptr(), dtype_code(pairs.dtype), ids.data_ptr(),
+                                  x.data_ptr(), ids.numel(), hidden, vocab, scale, buckets, mul_prev, mul_cur, last.data_ptr(),
+                                  last.stride(0), byref(batch), err.data_ptr(), stream), "embed_pairs")
 
 
 def rglru_conv(proj, bx, taps, cb, state, u, C: int, K: int, batch: BatchView, stream) -> None:

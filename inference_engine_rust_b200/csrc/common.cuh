@@ -32,11 +32,13 @@ enum : int { IERT_PAIR_HALF = 0, IERT_PAIR_INTERLEAVED = 1 };
 // One layer's keys and values in a paged cache group, plus the page tables of the group.
 //   k, v        : [n_pages][kv_heads][page_tokens][head_dim] of `dtype`
 //   page_table  : [n_slots][table_width]; logical block b of a sequence is entry
-//                 (b % ring_pages) of its row (ring_pages >= table_width means "no ring")
+//                 iert_table_entry(b) of its row: blocks below keep_pages stay where they are, the later ones go
+//                 round in the other ring_pages - keep_pages entries (ring_pages >= table_width means "no ring")
 //   window      : 0 = every earlier key is visible; W > 0 = the last W keys, the current
 //                 one included
 //   chunk       : C > 0 = only the keys of the position's own chunk of C positions (chunks are counted
 //                 from position 0 of the sequence); combines with a window (the later lower bound wins)
+//   keep        : the first `keep` positions of a sequence stay visible whatever window and chunk say
 struct IertKvView {
   void* k;
   void* v;
@@ -50,6 +52,8 @@ struct IertKvView {
   int dtype;
   int window;
   int chunk;
+  int keep;
+  int keep_pages;
 };
 
 // The first position that position `pos` sees under a window and a chunk rule (either may be 0 = none).
@@ -58,6 +62,40 @@ __host__ __device__ __forceinline__ int iert_first_visible(int pos, int window, 
   if (chunk > 0) { const int c = pos - pos % chunk; lo = lo > c ? lo : c; }
   return lo > 0 ? lo : 0;
 }
+
+// The entry of a sequence's page-table row that holds its logical block `blk`.
+__host__ __device__ __forceinline__ int iert_table_entry(const IertKvView& c, int blk) {
+  return blk < c.keep_pages ? blk : c.keep_pages + (blk - c.keep_pages) % (c.ring_pages - c.keep_pages);
+}
+
+// Is position `pos` of a sequence that ends a step with `final_len` positions written to the cache at all?  (Positions
+// that the ring would overwrite in the same step are not; kept pages are always written.)
+__host__ __device__ __forceinline__ bool iert_stays_cached(const IertKvView& c, int pos, int final_len) {
+  return pos >= final_len - (c.ring_pages - c.keep_pages) * c.page_tokens || pos < c.keep_pages * c.page_tokens;
+}
+
+// Blocks of `size` positions that lie below block `lo_blk` and hold kept first positions: a kernel visits them in front
+// of its own range [lo_blk, ...).
+__host__ __device__ __forceinline__ int iert_kept_blocks(int keep, int size, int lo_blk) {
+  const int n = (keep + size - 1) / size;
+  return n < lo_blk ? n : lo_blk;
+}
+
+// The pages (of `size` positions) that a one-token step at position `pos` walks: the `n_kept` first ones that hold kept
+// positions, then the pages of the window, [pg_lo, pos / size]; `n` in all, of which iert_walk_page() gives the i-th.
+// Position j is visible if j <= pos and (j >= j_min or j < keep).
+struct IertPageWalk {
+  int j_min, pg_lo, n_kept, n;
+};
+__device__ __forceinline__ IertPageWalk iert_page_walk(const IertKvView& c, int pos, int size) {
+  IertPageWalk w;
+  w.j_min = iert_first_visible(pos, c.window, c.chunk);
+  w.pg_lo = w.j_min / size;
+  w.n_kept = iert_kept_blocks(c.keep, size, w.pg_lo);
+  w.n = w.n_kept + pos / size + 1 - w.pg_lo;
+  return w;
+}
+__device__ __forceinline__ int iert_walk_page(const IertPageWalk& w, int i) { return i < w.n_kept ? i : w.pg_lo + i - w.n_kept; }
 
 // The sequences of one step.  All arrays live on the device.
 //   cu_q[n_seqs+1] : prefix sums of the tokens each sequence brings
@@ -226,7 +264,7 @@ __device__ __forceinline__ long long kv_row_offset(const IertKvView& c, int slot
                                                    int* err) {
   const int blk = pos / c.page_tokens;
   const int row = pos - blk * c.page_tokens;
-  const int entry = blk % c.ring_pages;
+  const int entry = iert_table_entry(c, blk);
   const int page = c.page_table[(long long)slot * c.table_width + entry];
   if (page < 0 || page >= c.n_pages) {
     if (err) atomicOr(err, IERT_ERR_PAGE_RANGE);

@@ -220,15 +220,15 @@ IERT_API int iert_rmsnorm(const float* x, const void* w, int w_dtype, void* out,
 // paged cache.  A block serves one token and a run of its heads (all of them when the step
 // has many tokens); heads [0, heads) are queries, the next kv_heads are keys, the last
 // kv_heads are values.  The token's cos/sin table is computed once per block.
-//   angle(pos, k) = pos * inv_freq[k] in fp32; (a, b) -> (a cos - b sin, a sin + b cos)
+//   angle(pos, k) = pos * inv_freq[k] in fp32; (a, b) -> (a cos - b sin, a sin + b cos) * rot_mul
 // Reference: src/ops/rope.rs:40-57 (rotation), src/layers/attention.rs:314-352 (order:
 // rotate, then append), :518-520 (decode position = cache length before the append).
 // A key or value is stored only if it can still be seen after this step: its position is
-// within the last ring_pages*page_tokens positions of its sequence.
+// within what the sequence's pages hold (see iert_stays_cached).
 template <typename T>
 __global__ void rope_kv_store_kernel(T* __restrict__ qkv, IertBatchView b, IertKvView c,
                                      const float* __restrict__ inv_freq, int heads,
-                                     int rotary_dim, int pairing, int write_cache,
+                                     int rotary_dim, float rot_mul, int pairing, int write_cache,
                                      int heads_per_block, int vec8, int* __restrict__ err) {
   extern __shared__ float cs[];                 // [rotary_dim / 2] cos, then [rotary_dim / 2] sin
   pdl_launch_dependents();     // the next kernel may start its preamble now
@@ -248,12 +248,12 @@ __global__ void rope_kv_store_kernel(T* __restrict__ qkv, IertBatchView b, IertK
   for (int k = threadIdx.x; k < half; k += blockDim.x) {   // the token's angles, once for all heads
     float sn, cs_;
     sincosf((float)pos * inv_freq[k], &sn, &cs_);
-    cs[k] = cs_;
-    cs[half + k] = sn;
+    cs[k] = cs_ * rot_mul;
+    cs[half + k] = sn * rot_mul;
   }
   __syncthreads();
   pdl_wait();                  // the projection is complete from here on
-  const bool store = write_cache && pos >= final_len - c.ring_pages * c.page_tokens;
+  const bool store = write_cache && iert_stays_cached(c, pos, final_len);
   T* row = qkv + (size_t)t * total_heads * hd;
   // this block's heads: [h0, h1) of [queries | keys | values]
   const int h0 = blockIdx.y * heads_per_block, h1 = min(total_heads, h0 + heads_per_block);
@@ -332,7 +332,7 @@ __global__ void rope_kv_store_kernel(T* __restrict__ qkv, IertBatchView b, IertK
 
 IERT_API int iert_rope_kv_store(void* qkv, int dtype, const IertBatchView* batch,
                                 const IertKvView* cache, const float* inv_freq, int heads,
-                                int rotary_dim, int pairing, int write_cache, int* err,
+                                int rotary_dim, float rot_mul, int pairing, int write_cache, int* err,
                                 cudaStream_t stream) {
   if (batch->n_tokens <= 0) return IERT_OK;
   if (rotary_dim < 0 || rotary_dim > cache->head_dim || (rotary_dim & 1) || cache->dtype != dtype)
@@ -351,9 +351,9 @@ IERT_API int iert_rope_kv_store(void* qkv, int dtype, const IertBatchView* batch
   const int vec8 = dtype == IERT_BF16 && hd % 8 == 0 && rotary_dim % (pairing == IERT_PAIR_HALF ? 16 : 8) == 0 &&
                    (((uintptr_t)qkv | (uintptr_t)cache->k | (uintptr_t)cache->v) & 15) == 0;
   if (dtype == IERT_F32)
-    launch_dep(rope_kv_store_kernel<float>, grid, dim3(threads), smem, stream, (float*)qkv, *batch, *cache, inv_freq, heads, rotary_dim, pairing, write_cache, heads_per_block, 0, err);
+    launch_dep(rope_kv_store_kernel<float>, grid, dim3(threads), smem, stream, (float*)qkv, *batch, *cache, inv_freq, heads, rotary_dim, rot_mul, pairing, write_cache, heads_per_block, 0, err);
   else if (dtype == IERT_BF16)
-    launch_dep(rope_kv_store_kernel<__nv_bfloat16>, grid, dim3(threads), smem, stream, (__nv_bfloat16*)qkv, *batch, *cache, inv_freq, heads, rotary_dim, pairing, write_cache, heads_per_block, vec8, err);
+    launch_dep(rope_kv_store_kernel<__nv_bfloat16>, grid, dim3(threads), smem, stream, (__nv_bfloat16*)qkv, *batch, *cache, inv_freq, heads, rotary_dim, rot_mul, pairing, write_cache, heads_per_block, vec8, err);
   else
     return IERT_BAD_ARGUMENT;
   return iert_check_launch("rope_kv_store");

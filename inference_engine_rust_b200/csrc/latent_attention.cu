@@ -168,8 +168,11 @@ latent_attention_decode_kernel(const T* __restrict__ q, long long ldq, const T* 
 #pragma unroll
   for (int i = 0; i < MAX_PER_THREAD; ++i) acc[i] = 0.f;
   const T* cache = (const T*)kv.k;
-  for (int j0 = 0; j0 <= pos; j0 += THREADS) {
-    const int j = j0 + threadIdx.x;
+  const int j_min = iert_first_visible(pos, kv.window, kv.chunk), n_keep = min(kv.keep, j_min);
+  const int n_keys = n_keep + pos - j_min + 1;       // visible keys, numbered i: kept first positions, then [j_min, pos]
+  auto key_of = [&](int i) { return i < n_keep ? i : j_min + i - n_keep; };
+  for (int i0 = 0; i0 < n_keys; i0 += THREADS) {
+    const int j = key_of(i0 + threadIdx.x);
     float sc = -INFINITY;
     if (j <= pos) {
       const long long off = kv_row_offset(kv, slot, j, 0, err);
@@ -181,7 +184,7 @@ latent_attention_decode_kernel(const T* __restrict__ q, long long ldq, const T* 
       }
     }
     const float alpha = softmax_chunk(sc, m, l, p_s, scratch);
-    const int n_in = min(THREADS, pos - j0 + 1);
+    const int n_in = min(THREADS, n_keys - i0);
 #pragma unroll
     for (int i = 0; i < MAX_PER_THREAD; ++i) {
       const int r = threadIdx.x + i * THREADS;
@@ -190,7 +193,7 @@ latent_attention_decode_kernel(const T* __restrict__ q, long long ldq, const T* 
       for (int jj = 0; jj < n_in; ++jj) {
         const float pj = p_s[jj];
         if (pj == 0.f) continue;
-        const long long off = kv_row_offset(kv, slot, j0 + jj, 0, nullptr);
+        const long long off = kv_row_offset(kv, slot, key_of(i0 + jj), 0, nullptr);
         if (off < 0) continue;
         a = fmaf(pj, to_f32(cache[off + r]), a);
       }
@@ -215,70 +218,137 @@ latent_attention_decode_kernel(const T* __restrict__ q, long long ldq, const T* 
   }
 }
 
-// The step's rows of latent attention with a rotated part, from one fp32 projection row per token
-//   x = [ q: H heads of (D unrotated | R rotated) | down: rank latent numbers | R rotated key numbers | H gate logits ]
-// to what the attention kernels read:
-//   c_ext [T, rank + R]   RMS-normed latent (plain weight, eps inside the root) | rotated key part; also the cache row
-//   q_out [T, H, q_head]  per head (D unrotated | R rotated | zeros up to q_head)
-//   gate_out [T, H]       sigmoid(gate logit) * out_scale  (fp32), if the layer has a gate
-// Angles are position * inv_freq[i] in fp32 with the precise sine and cosine; pairs are neighbours (2i, 2i+1) or
-// halves (i, i + R/2).  One block per token; all arithmetic fp32, one rounding at the store.
-template <typename T>
-__global__ void latent_prep_kernel(const float* __restrict__ x, long long ldx, int H, int D, int R, int rank,
-                                   const float* __restrict__ wkv, float eps, const float* __restrict__ inv_freq, int pairing,
-                                   int has_gate, float out_scale, T* __restrict__ c_ext, T* __restrict__ q_out, long long ldq,
-                                   int q_head, float* __restrict__ gate_out, IertBatchView b, IertKvView kv, int store,
-                                   int* __restrict__ err) {
+// The step's rows of latent attention with a rotated part, from fp32 projection rows to what the attention kernels read.
+// Each of the four pieces is there or not (null), so that one launch does what its inputs allow:
+//   down  rank latent numbers | R rotated key numbers  ->  c_ext [T, rank + R] = RMS-normed latent (plain weight, eps
+//         inside the root) | rotated key part; also the cache row
+//   q     H heads of (D unrotated | R rotated)  ->  q_out, per head (D unrotated | R rotated | zeros up to q_head)
+//   dq    q_rank numbers of a query latent  ->  cq = RMS-normed (plain weight)
+//   glog  H gate logits  ->  gate_out [T, H] = sigmoid * out_scale (fp32)
+// Angles are position * inv_freq[i] in fp32 with the precise sine and cosine, times `rot_mul`; pairs are neighbours
+// (2i, 2i+1) or halves (i, i + R/2).  One block per token; all arithmetic fp32, one rounding at the store.
+struct LatentPrep {
+  const float* q; const float* down; const float* dq; const float* glog;
+  long long ldq_in, ld_down, ld_dq, ld_glog;
+  int H, D, R, rank, q_rank, q_head, pairing, store;
+  const float* wkv; const float* wq; const float* inv_freq;
+  float eps, rot_mul, out_scale;
+  void* c_ext; void* q_out; void* cq;
+  long long ldq;
+  float* gate_out;
+};
+
+__device__ __forceinline__ void latent_put4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void latent_put4(__nv_bfloat16* p, const float4& v) {
+  uint2 w;
+  *reinterpret_cast<__nv_bfloat162*>(&w.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&w.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = w;
+}
+
+// VEC: the queries in groups of four numbers (16-byte loads): D, R / 2, q_head and the row strides are multiples of 4
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+latent_prep_kernel(LatentPrep a, IertBatchView b, IertKvView kv, int* __restrict__ err) {
+  extern __shared__ float cs[];           // [R / 2] cos, [R / 2] sin
   __shared__ float scratch[33];
-  pdl_wait();
+  pdl_launch_dependents();
   const int t = blockIdx.x;
   const int s = sequence_of_token(b, t);
   const int slot = s >= 0 ? b.slot_ids[s] : -1;
-  T* qrow = q_out + (size_t)t * ldq;
+  T* qrow = a.q ? (T*)a.q_out + (size_t)t * a.ldq : nullptr;
+  T* crow = a.down ? (T*)a.c_ext + (size_t)t * (a.rank + a.R) : nullptr;
+  T* cqrow = a.dq ? (T*)a.cq + (size_t)t * a.q_rank : nullptr;
   if (slot < 0) {                       // padding: rows of zeros, nothing stored
-    for (int i = threadIdx.x; i < H * q_head; i += blockDim.x) qrow[i] = from_f32<T>(0.f);
-    for (int i = threadIdx.x; i < rank + R; i += blockDim.x) c_ext[(size_t)t * (rank + R) + i] = from_f32<T>(0.f);
-    if (has_gate) for (int i = threadIdx.x; i < H; i += blockDim.x) gate_out[(size_t)t * H + i] = 0.f;
+    pdl_wait();
+    if (qrow) for (int i = threadIdx.x; i < a.H * a.q_head; i += blockDim.x) qrow[i] = from_f32<T>(0.f);
+    if (crow) for (int i = threadIdx.x; i < a.rank + a.R; i += blockDim.x) crow[i] = from_f32<T>(0.f);
+    if (cqrow) for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cqrow[i] = from_f32<T>(0.f);
+    if (a.glog) for (int i = threadIdx.x; i < a.H; i += blockDim.x) a.gate_out[(size_t)t * a.H + i] = 0.f;
     return;
   }
   const int pos = b.pos0[s] + (t - b.cu_q[s]);
-  const float* row = x + (size_t)t * ldx;
-  const float* down = row + (size_t)H * (D + R);
-  const float* glog = down + rank + R;
-  const int half = R / 2;
-  // the rotated partner and sign of element i of a rotated part: out = v[i] cos - v[partner] sin for the first of a pair
+  const int R = a.R, D = a.D, half = R / 2;
+  for (int k = threadIdx.x; k < half; k += blockDim.x) {
+    float sn, co;
+    sincosf((float)pos * a.inv_freq[k], &sn, &co);
+    cs[k] = co * a.rot_mul;
+    cs[half + k] = sn * a.rot_mul;
+  }
+  pdl_wait();
+  __syncthreads();
+  // element i of a rotated part: out = v[i] cos - v[partner] sin for the first of a pair, v[i] cos + v[partner] sin else
   auto rotated = [&](const float* v, int i) -> float {
     int k, first;
-    if (pairing == IERT_PAIR_INTERLEAVED) { k = i >> 1; first = !(i & 1); }
+    if (a.pairing == IERT_PAIR_INTERLEAVED) { k = i >> 1; first = !(i & 1); }
     else { k = i < half ? i : i - half; first = i < half; }
-    const int other = pairing == IERT_PAIR_INTERLEAVED ? (i ^ 1) : (first ? i + half : i - half);
-    float sn, cs;
-    sincosf((float)pos * inv_freq[k], &sn, &cs);
-    return first ? v[i] * cs - v[other] * sn : v[i] * cs + v[other] * sn;
+    const int other = a.pairing == IERT_PAIR_INTERLEAVED ? (i ^ 1) : (first ? i + half : i - half);
+    return first ? v[i] * cs[k] - v[other] * cs[half + k] : v[i] * cs[k] + v[other] * cs[half + k];
   };
-  for (int i = threadIdx.x; i < H * q_head; i += blockDim.x) {
-    const int h = i / q_head, d = i - h * q_head;
-    const float* qh = row + (size_t)h * (D + R);
-    float v = 0.f;
-    if (d < D) v = qh[d];
-    else if (d < D + R) v = rotated(qh + D, d - D);
-    qrow[i] = from_f32<T>(v);
+  if (qrow) {
+    const float* row = a.q + (size_t)t * a.ldq_in;
+    if (VEC) {
+      const int per = a.q_head / 4;
+      for (int i = threadIdx.x; i < a.H * per; i += blockDim.x) {
+        const int h = i / per, d = 4 * (i - h * per);
+        const float* qh = row + (size_t)h * (D + R);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d < D + R) v = *reinterpret_cast<const float4*>(qh + d);
+        if (d >= D && d < D + R) {
+          const int e = d - D;
+          if (a.pairing == IERT_PAIR_INTERLEAVED) {
+            const int k = e >> 1;
+            v = make_float4(v.x * cs[k] - v.y * cs[half + k], v.y * cs[k] + v.x * cs[half + k],
+                            v.z * cs[k + 1] - v.w * cs[half + k + 1], v.w * cs[k + 1] + v.z * cs[half + k + 1]);
+          } else {
+            const bool first = e < half;
+            const int k = first ? e : e - half;
+            const float4 o = *reinterpret_cast<const float4*>(qh + D + (first ? e + half : e - half));
+            const float sg = first ? -1.f : 1.f;
+            v = make_float4(v.x * cs[k] + sg * o.x * cs[half + k], v.y * cs[k + 1] + sg * o.y * cs[half + k + 1],
+                            v.z * cs[k + 2] + sg * o.z * cs[half + k + 2], v.w * cs[k + 3] + sg * o.w * cs[half + k + 3]);
+          }
+        }
+        latent_put4(qrow + h * a.q_head + d, v);
+      }
+    } else {
+      for (int i = threadIdx.x; i < a.H * a.q_head; i += blockDim.x) {
+        const int h = i / a.q_head, d = i - h * a.q_head;
+        const float* qh = row + (size_t)h * (D + R);
+        float v = 0.f;
+        if (d < D) v = qh[d];
+        else if (d < D + R) v = rotated(qh + D, d - D);
+        qrow[i] = from_f32<T>(v);
+      }
+    }
   }
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) ss = fmaf(down[i], down[i], ss);
-  const float rk = 1.0f / sqrtf(block_sum(ss, scratch) / (float)rank + eps);
-  T* dst = nullptr;
-  if (store && pos >= b.pos0[s] + (b.cu_q[s + 1] - b.cu_q[s]) - kv.ring_pages * kv.page_tokens) {
-    const long long off = kv_row_offset(kv, slot, pos, 0, err);
-    if (off >= 0) dst = (T*)kv.k + off;
+  if (cqrow) {
+    const float* v = a.dq + (size_t)t * a.ld_dq;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) ss = fmaf(v[i], v[i], ss);
+    const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)a.q_rank + a.eps);
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cqrow[i] = from_f32<T>(v[i] * r * a.wq[i]);
   }
-  for (int i = threadIdx.x; i < rank + R; i += blockDim.x) {
-    const T v = from_f32<T>(i < rank ? down[i] * rk * wkv[i] : rotated(down + rank, i - rank));
-    c_ext[(size_t)t * (rank + R) + i] = v;
-    if (dst) dst[i] = v;
+  if (crow) {
+    const float* down = a.down + (size_t)t * a.ld_down;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < a.rank; i += blockDim.x) ss = fmaf(down[i], down[i], ss);
+    const float rk = 1.0f / sqrtf(block_sum(ss, scratch) / (float)a.rank + a.eps);
+    T* dst = nullptr;
+    if (a.store && iert_stays_cached(kv, pos, b.pos0[s] + (b.cu_q[s + 1] - b.cu_q[s]))) {
+      const long long off = kv_row_offset(kv, slot, pos, 0, err);
+      if (off >= 0) dst = (T*)kv.k + off;
+    }
+    for (int i = threadIdx.x; i < a.rank + R; i += blockDim.x) {
+      const T v = from_f32<T>(i < a.rank ? down[i] * rk * a.wkv[i] : rotated(down + a.rank, i - a.rank));
+      crow[i] = v;
+      if (dst) dst[i] = v;
+    }
   }
-  if (has_gate)
-    for (int i = threadIdx.x; i < H; i += blockDim.x) gate_out[(size_t)t * H + i] = out_scale / (1.0f + expf(-glog[i]));
+  if (a.glog) {
+    const float* g = a.glog + (size_t)t * a.ld_glog;
+    for (int i = threadIdx.x; i < a.H; i += blockDim.x) a.gate_out[(size_t)t * a.H + i] = a.out_scale / (1.0f + expf(-g[i]));
+  }
 }
 
 // out[t, h, :V] = attn[t, h, :V] * gate[t, h]: drops the padding of heads of `head` numbers and applies the gate.
@@ -376,26 +446,37 @@ IERT_API int iert_latent_attention_decode(const void* q, long long ldq, const vo
   return iert_check_launch("latent_attention_decode");
 }
 
-// x: fp32 [T, ldx] = q [H * (D + R)] | latent [rank] | rotated key part [R] | gate logits [H] (if has_gate).
-// c_ext [T, rank + R], q_out [T, H * q_head] with row stride ldq (q_head >= D + R) in `dtype`; gate_out fp32 [T, H]; inv_freq fp32 [R / 2].
-// With `store` the rows of c_ext also go to the cache (kv_heads 1, head_dim rank + R, keys only).
-IERT_API int iert_latent_prep(const float* x, long long ldx, int H, int D, int R, int rank, const float* wkv, float eps,
-                              const float* inv_freq, int pairing, int has_gate, float out_scale, void* c_ext, void* q_out,
-                              long long ldq, int q_head, float* gate_out, int dtype, const IertBatchView* batch, const IertKvView* kv,
-                              int store, int* err, cudaStream_t stream) {
+// See LatentPrep: the fp32 inputs q [T, H * (D + R)], down [T, rank + R], dq [T, q_rank] and glog [T, H] are each there or
+// null, with row strides of their own.  c_ext [T, rank + R], q_out [T, H * q_head] with row stride ldq (q_head >= D + R)
+// and cq [T, q_rank] in `dtype`; gate_out fp32 [T, H]; inv_freq fp32 [R / 2].  With `store` the rows of c_ext also go to the
+// cache (kv_heads 1, head_dim rank + R, keys only).
+IERT_API int iert_latent_prep(const float* q, long long ldq_in, const float* down, long long ld_down, const float* dq,
+                              long long ld_dq, const float* glog, long long ld_glog, int H, int D, int R, int rank, int q_rank,
+                              const float* wkv, const float* wq, float eps, const float* inv_freq, float rot_mul, int pairing,
+                              float out_scale, void* c_ext, void* q_out, long long ldq, int q_head, void* cq, float* gate_out,
+                              int dtype, const IertBatchView* batch, const IertKvView* kv, int store, int* err,
+                              cudaStream_t stream) {
   if (batch->n_tokens <= 0) return IERT_OK;
-  if (H <= 0 || D < 0 || R < 0 || (R & 1) || rank <= 0 || q_head < D + R || ldq < (long long)H * q_head || (R > 0 && !inv_freq) || (has_gate && !gate_out) ||
-      (pairing != IERT_PAIR_HALF && pairing != IERT_PAIR_INTERLEAVED) ||
-      (store && (kv->head_dim != rank + R || kv->kv_heads != 1 || kv->dtype != dtype)))
+  if (H <= 0 || D < 0 || R < 0 || (R & 1) || rank <= 0 || (R > 0 && !inv_freq) || (glog && !gate_out) ||
+      (pairing != IERT_PAIR_HALF && pairing != IERT_PAIR_INTERLEAVED) || R > 8192 ||
+      (q && (!q_out || q_head < D + R || ldq < (long long)H * q_head)) || (down && (!c_ext || !wkv)) ||
+      (dq && (!cq || !wq || q_rank <= 0)) ||
+      (down && store && (kv->head_dim != rank + R || kv->kv_heads != 1 || kv->dtype != dtype)))
     return IERT_BAD_ARGUMENT;
-  if (dtype == IERT_F32)
-    launch_dep(latent_prep_kernel<float>, dim3(batch->n_tokens), dim3(256), 0, stream, x, ldx, H, D, R, rank, wkv, eps, inv_freq,
-               pairing, has_gate, out_scale, (float*)c_ext, (float*)q_out, ldq, q_head, gate_out, *batch, *kv, store, err);
-  else if (dtype == IERT_BF16)
-    launch_dep(latent_prep_kernel<__nv_bfloat16>, dim3(batch->n_tokens), dim3(256), 0, stream, x, ldx, H, D, R, rank, wkv, eps,
-               inv_freq, pairing, has_gate, out_scale, (__nv_bfloat16*)c_ext, (__nv_bfloat16*)q_out, ldq, q_head, gate_out, *batch,
-               *kv, store, err);
+  LatentPrep a = {q, down, dq, glog, ldq_in, ld_down, ld_dq, ld_glog, H, D, R, rank, q_rank, q_head, pairing, store, wkv, wq,
+                  inv_freq, eps, rot_mul, out_scale, c_ext, q_out, cq, ldq, gate_out};
+  const int elt = dtype == IERT_F32 ? 4 : 2;
+  const bool vec = q && D % 4 == 0 && (R / 2) % 4 == 0 && q_head % 4 == 0 && ldq % 4 == 0 && ldq_in % 4 == 0 && ((uintptr_t)q & 15) == 0 &&
+                   ((uintptr_t)q_out % (4 * elt)) == 0;
+#define GO(T)                                                                                                                        \
+  do {                                                                                                                               \
+    if (vec) launch_dep(latent_prep_kernel<T, true>, dim3(batch->n_tokens), dim3(256), R * sizeof(float), stream, a, *batch, *kv, err); \
+    else launch_dep(latent_prep_kernel<T, false>, dim3(batch->n_tokens), dim3(256), R * sizeof(float), stream, a, *batch, *kv, err);    \
+  } while (0)
+  if (dtype == IERT_F32) GO(float);
+  else if (dtype == IERT_BF16) GO(__nv_bfloat16);
   else return IERT_BAD_ARGUMENT;
+#undef GO
   return iert_check_launch("latent_prep");
 }
 

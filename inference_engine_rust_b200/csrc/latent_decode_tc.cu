@@ -6,7 +6,8 @@
 //
 // which is multi-query attention whose keys and values are the same rows.  W_uv is applied to L at the
 // end, once per head.  Three kernels:
-//   latent_absorb_q       qa [T, Hpad, rank] bf16 from q and W_uk (rows of padding heads are zero)
+//   latent_absorb_q       qa [T, Hpad, rank] bf16 from q and W_uk (rows of padding heads are zero); q either in bf16 with
+//                         its rotated part turned already, or the fp32 projection itself, turned on the way
 //   latent_decode_tc      a CTA takes (sequence, a run of 64-key tiles, up to 32 heads): the tile of C comes
 //                         into shared memory once (cp.async) and serves both products; warp w forms the
 //                         scores of keys 16w..16w+15 of the tile for all the CTA's heads, the warps agree on
@@ -14,6 +15,7 @@
 //                         rank columns of L (its accumulators).  Partial (max, sum, L) per run go to scratch.
 //   latent_decode_merge   merges the runs in order, adds the sink's term exp(sink - M) to the denominator,
 //                         and multiplies by W_uv: out [T, H*V].
+// A window, a chunk or kept first positions of the cache view choose which pages are walked and which rows count.
 // Sizes: rank a multiple of 32 up to 512, pages of 64 positions, a bf16 cache.  Anything else is refused
 // (IERT_BAD_ARGUMENT) and the caller runs the plain kernel.
 #include "common.cuh"
@@ -40,12 +42,16 @@ __device__ __forceinline__ uint32_t lds32(const __nv_bfloat16* p) { return *rein
 // through shared memory in a fixed order.
 constexpr int ABSORB_THREADS = 256;
 
+// TQ float: q is the projection as it stands, and the R last numbers of a head are turned here (inv_freq, rot_mul, pairing).
+template <typename TQ>
 __global__ void __launch_bounds__(ABSORB_THREADS)
-latent_absorb_q_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, const __nv_bfloat16* __restrict__ w_uk,
-                       __nv_bfloat16* __restrict__ qa, int H, int Hpad, int D, int R, int rank) {
+latent_absorb_q_kernel(const TQ* __restrict__ q, long long ldq, const __nv_bfloat16* __restrict__ w_uk,
+                       __nv_bfloat16* __restrict__ qa, int H, int Hpad, int D, int R, int rank, const float* __restrict__ inv_freq,
+                       float rot_mul, int pairing, IertBatchView b) {
   extern __shared__ float sm_q[];
   float* q_s = sm_q;                    // [D]
   float* part = sm_q + D;               // [4][rank]
+  pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
   __nv_bfloat16* dst = qa + ((size_t)t * Hpad + h) * (rank + R);
@@ -53,9 +59,23 @@ latent_absorb_q_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, const
     for (int r = threadIdx.x; r < rank + R; r += blockDim.x) dst[r] = __float2bfloat16_rn(0.f);
     return;
   }
-  const __nv_bfloat16* qh = q + (size_t)t * ldq + (size_t)h * (D + R);
-  for (int d = threadIdx.x; d < D; d += blockDim.x) q_s[d] = __bfloat162float(qh[d]);
-  for (int i = threadIdx.x; i < R; i += blockDim.x) dst[rank + i] = qh[D + i];      // the rotated part passes as it is
+  const TQ* qh = q + (size_t)t * ldq + (size_t)h * (D + R);
+  for (int d = threadIdx.x; d < D; d += blockDim.x) q_s[d] = to_f32(qh[d]);
+  if (sizeof(TQ) == 4) {                // one token per sequence: token t is sequence t's
+    const int half = R / 2, pos = b.pos0[t];
+    for (int k = threadIdx.x; k < half; k += blockDim.x) {
+      const int i0 = pairing == IERT_PAIR_INTERLEAVED ? 2 * k : k, i1 = pairing == IERT_PAIR_INTERLEAVED ? 2 * k + 1 : k + half;
+      const float u = to_f32(qh[D + i0]), v = to_f32(qh[D + i1]);
+      float sn, co;
+      sincosf((float)pos * inv_freq[k], &sn, &co);
+      sn *= rot_mul;
+      co *= rot_mul;
+      dst[rank + i0] = __float2bfloat16_rn(u * co - v * sn);
+      dst[rank + i1] = __float2bfloat16_rn(v * co + u * sn);
+    }
+  } else {
+    for (int i = threadIdx.x; i < R; i += blockDim.x) dst[rank + i] = __float2bfloat16_rn(to_f32(qh[D + i]));   // turned already
+  }
   __syncthreads();
   const int grp = threadIdx.x >> 6, lane64 = threadIdx.x & 63;
   const int d_lo = grp * ((D + 3) / 4), d_hi = min(D, d_lo + (D + 3) / 4);
@@ -95,12 +115,14 @@ latent_decode_tc_kernel(const __nv_bfloat16* __restrict__ qa, IertBatchView b, I
   __nv_bfloat16* p_s = c_s + BK * ldc;                               // [MT*16][PLD]
   float* wmax = reinterpret_cast<float*>(p_s + MT * 16 * PLD);       // [4][MT*16]
   float* wsum = wmax + 4 * MT * 16;                                  // [4][MT*16]
+  pdl_launch_dependents();
   pdl_wait();
   const int s = blockIdx.x, split = blockIdx.y, rows0 = blockIdx.z * MT * 16;
   const int slot = b.slot_ids[s];
   if (slot < 0) return;
-  const int n_keys = b.pos0[s] + 1;                  // one token per sequence: its own row is in the cache
-  const int n_tiles = (n_keys + BK - 1) / BK;
+  const int pos = b.pos0[s];                         // one token per sequence: its own row is in the cache
+  const IertPageWalk walk = iert_page_walk(kv, pos, BK);
+  const int n_tiles = walk.n;
   const int t_lo = (int)((long long)split * n_tiles / splits), t_hi = (int)((long long)(split + 1) * n_tiles / splits);
   const size_t part_row0 = ((size_t)s * splits + split) * Hpad + rows0;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
@@ -127,15 +149,17 @@ latent_decode_tc_kernel(const __nv_bfloat16* __restrict__ qa, IertBatchView b, I
 
   for (int tile = t_lo; tile < t_hi; ++tile) {
     __syncthreads();                                 // the tile before is no longer read (and qa_s is written)
-    const int page = kv.page_table[(size_t)slot * kv.table_width + (tile % kv.ring_pages)];
+    const int pg = iert_walk_page(walk, tile);
+    const int page = kv.page_table[(size_t)slot * kv.table_width + iert_table_entry(kv, pg)];
     const bool page_ok = page >= 0 && page < kv.n_pages;
     if (!page_ok && tid == 0) atomicOr(err, IERT_ERR_PAGE_RANGE);
     const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(kv.k) + (size_t)(page_ok ? page : 0) * BK * width;
-    const int valid = page_ok ? min(BK, n_keys - tile * BK) : 0;     // rows beyond hold other sequences' leftovers
+    const int valid = page_ok ? min(BK, pos + 1 - pg * BK) : 0;      // rows beyond hold other sequences' leftovers
+    const int first = walk.j_min - pg * BK, kept = kv.keep - pg * BK;   // rows in front of the window count if they are kept
     for (int i = tid; i < BK * chunks; i += THREADS) {
       const int r = i / chunks, c = i - r * chunks;
       __nv_bfloat16* dst = c_s + r * ldc + c * 8;
-      if (r < valid)
+      if (r < valid && (r >= first || r < kept))
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src + (size_t)r * width + c * 8));
       else
         *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
@@ -176,7 +200,7 @@ latent_decode_tc_kernel(const __nv_bfloat16* __restrict__ qa, IertBatchView b, I
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             const int j = warp * 16 + nt * 8 + 2 * t4 + e;
-            const float v = j < valid ? sc[mt][nt][half * 2 + e] * scale : -INFINITY;
+            const float v = (j < valid && (j >= first || j < kept)) ? sc[mt][nt][half * 2 + e] * scale : -INFINITY;
             sc[mt][nt][half * 2 + e] = v;
             mx = fmaxf(mx, v);
           }
@@ -195,7 +219,7 @@ latent_decode_tc_kernel(const __nv_bfloat16* __restrict__ qa, IertBatchView b, I
 #pragma unroll
         for (int w = 0; w < 4; ++w) m_new = fmaxf(m_new, wmax[w * MT * 16 + row]);
         alpha[mt][half] = m_run[mt][half] == -INFINITY ? 0.f : expf(m_run[mt][half] - m_new);
-        m_run[mt][half] = m_new;                     // finite: every tile of a run holds at least one key
+        m_run[mt][half] = m_new;                     // finite: every page of the walk holds at least one visible key
         float sum = 0.f;
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
@@ -271,6 +295,7 @@ latent_decode_merge_kernel(const float* __restrict__ part_m, const float* __rest
   extern __shared__ float sm[];
   float* lat = sm;                 // [rank]
   float* wgt = sm + rank;          // [64]
+  pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
   T* o = out + ((size_t)t * H + h) * V;
@@ -367,11 +392,12 @@ IERT_API int iert_latent_decode_tc_plan(int n_seqs, int H, int table_width, int*
   return IERT_OK;
 }
 
-// q [T, ldq] bf16 (H*(D+R) per token, one token per sequence: per head D unrotated and R rotated numbers); the cache's
+// q [T, ldq] (H*(D+R) per token, one token per sequence: per head D unrotated and R rotated numbers), bf16 with the rotated
+// numbers turned already, or with q_f32 != 0 fp32 as projected (turned here by inv_freq, rot_mul and pairing); the cache's
 // rows are rank + R wide (latent | rotated key part); w_uk [H*D, rank], w_uv [H*V, rank] bf16 row-major; gate: fp32 [T, H]
 // or null.  qa: scratch bf16 [T, Hpad, rank + R]; part_m, part_l: fp32 [T, splits, Hpad]; part_acc: fp32 [T, splits, Hpad, rank];
 // out bf16 [T, H*V].  Hpad and splits as iert_latent_decode_tc_plan gives them.
-IERT_API int iert_latent_attention_decode_tc(const void* q, long long ldq, const void* w_uk, const void* w_uv, void* out,
+IERT_API int iert_latent_attention_decode_tc(const void* q, int q_f32, long long ldq, const float* inv_freq, float rot_mul, int pairing, const void* w_uk, const void* w_uv, void* out,
                                              const IertBatchView* batch, const IertKvView* kv, int H, int D, int R, int V,
                                              float scale, const float* sink, const float* gate, int Hpad, int splits,
                                              void* qa, float* part_m, float* part_l, float* part_acc, int* err,
@@ -380,7 +406,7 @@ IERT_API int iert_latent_attention_decode_tc(const void* q, long long ldq, const
   if (T <= 0) return IERT_OK;
   if (T != batch->n_seqs || kv->dtype != IERT_BF16 || kv->kv_heads != 1 || kv->page_tokens != BK || rank % 32 || R < 0 ||
       R % 16 || width > 640 || rank < 32 || rank > MAX_NTW * 32 || H <= 0 || Hpad % 16 || Hpad < H || Hpad > 65535 || splits < 1 || splits > 64 ||
-      D <= 0 || D > 8192 || V <= 0 || (ldq % 8) || ((uintptr_t)q & 15))
+      D <= 0 || D > 8192 || V <= 0 || (q_f32 && R > 0 && !inv_freq))
     return IERT_BAD_ARGUMENT;
   const int mt = Hpad % 32 == 0 ? 2 : 1;
   const size_t smem = decode_smem(mt, width);
@@ -394,8 +420,14 @@ IERT_API int iert_latent_attention_decode_tc(const void* q, long long ldq, const
     }
     configured = true;
   }
-  launch_dep(latent_absorb_q_kernel, dim3(T, Hpad), dim3(ABSORB_THREADS), (size_t)(D + 4 * rank) * sizeof(float), stream,
-             (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)w_uk, (__nv_bfloat16*)qa, H, Hpad, D, R, rank);
+  const size_t absorb_smem = (size_t)(D + 4 * rank) * sizeof(float);
+  if (q_f32)
+    launch_dep(latent_absorb_q_kernel<float>, dim3(T, Hpad), dim3(ABSORB_THREADS), absorb_smem, stream, (const float*)q, ldq,
+               (const __nv_bfloat16*)w_uk, (__nv_bfloat16*)qa, H, Hpad, D, R, rank, inv_freq, rot_mul, pairing, *batch);
+  else
+    launch_dep(latent_absorb_q_kernel<__nv_bfloat16>, dim3(T, Hpad), dim3(ABSORB_THREADS), absorb_smem, stream,
+               (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)w_uk, (__nv_bfloat16*)qa, H, Hpad, D, R, rank, inv_freq, rot_mul,
+               pairing, *batch);
   dim3 grid(T, splits, Hpad / (mt * 16));
   if (mt == 2)
     launch_dep(latent_decode_tc_kernel<2>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16*)qa, *batch, *kv, Hpad, R,

@@ -53,7 +53,7 @@ qk_prep_kernel(const float* __restrict__ proj, long long ld, T* __restrict__ qkv
     cs[half + k] = sn;
   }
   pdl_wait();
-  const bool store = write_cache && pos >= final_len - c.ring_pages * c.page_tokens;
+  const bool store = write_cache && iert_stays_cached(c, pos, final_len);
   const float* pr = proj + (size_t)t * ld;
   T* out = qkv + (size_t)t * (qd + 2 * kd);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_heads = heads + nkv;

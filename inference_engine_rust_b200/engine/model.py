@@ -163,12 +163,22 @@ class Model:
 
     # ---- cache ----------------------------------------------------------------------------
     def cache_requests(self) -> Dict[int, CacheRequest]:
-        """What each cache-writing schedule entry asks of the cache, keyed by its position."""
+        """What each cache-writing schedule entry asks of the cache, keyed by its position, and what the step inputs ask
+        (keys below 0)."""
         out = {}
         for pos, e in enumerate(self.spec.schedule):
             if e.writes_cache:
                 out[pos] = self._layer_parts[e.layer][1].cache_request()
+        for i, (part, _) in enumerate(self.inputs):
+            request = getattr(part, "cache_request", lambda: None)()
+            if request is not None:
+                out[self._input_key(i)] = request
         return out
+
+    @staticmethod
+    def _input_key(i: int) -> int:
+        """Under which key the cache keeps what the i-th step input asked for (the schedule's entries count from 0)."""
+        return -1 - i
 
     def graph_safe(self) -> bool:
         """True when every part declares `graph_safe`: its forward reads the step's sequences
@@ -231,10 +241,17 @@ class Model:
         if request is not None:
             from ..parts.norm import honour
             ahead, finish = honour(request, x, ctx, "embed", 1)
-        B.embed_gather(self.embedding, tokens, x, spec.embedding_scale, rt.err, ctx.stream, ahead=ahead)
+        embeds = bool(self.inputs) and getattr(self.inputs[0][0], "embeds", False)
+        if not embeds:
+            B.embed_gather(self.embedding, tokens, x, spec.embedding_scale, rt.err, ctx.stream, ahead=ahead)
         ctx.rows_ahead = finish() if finish is not None else None
-        for part, _ in self.inputs:
-            part.prepare(tokens, x, ctx)
+        for i, (part, _) in enumerate(self.inputs):
+            ctx.input_view = cache.layer_view(self._input_key(i))
+            if i == 0 and embeds:
+                part.embed(self.embedding, tokens, x, spec.embedding_scale, ctx)
+            else:
+                part.prepare(tokens, x, ctx)
+        ctx.input_view = None
         S = spec.residual_streams
         rows = x
         if S is not None:

@@ -6,7 +6,7 @@ learns which model it belongs to.  Adding a part means registering a class under
 kind; the configuration then names that kind for the layers that use it.
 
     norm      Norm(spec, hidden_size, rt)        .forward(x_f32, out, ctx, rows_idx=None, rows=None)
-    position  PositionEncoding(spec, head_dim, rt)   .encode(qkv, ctx, heads, kv_heads)   [.rotary_constants()]
+    position  PositionEncoding(spec, head_dim, rt)   .encode(qkv, ctx, heads, kv_heads)   [.rotary_constants(), .scaled_rotary_constants()]
     mixer     Mixer(spec, rt)                    .forward(xn, residual, ctx, cache_view, writes_cache)
     ffn       FeedForward(spec, rt)              .forward(xn, residual, ctx)
     block     Block(layer_spec, norm1, mixer, norm2, ffn, rt[, extra_norms={role: norm}])   .forward(x, ctx, cache_view, writes_cache)
@@ -155,7 +155,8 @@ class StepContext:
                                                    # applied next to the residual rows it writes
     rows_ahead: Optional[LazyInput] = None         # set by whoever honoured `norm_ahead`: that norm's lazy result
     next_block: object = None                      # the block that runs after the current one (None: the last)
-    shared: dict = field(default_factory=dict)     # what the model's step inputs published for the blocks, by name
+    shared: dict = field(default_factory=dict)     # what step inputs and mixers published for later blocks of the step, by name
+    input_view: object = None                      # while a step input runs: the view of what it asked of the cache (or None)
     slot_ids_dev: Optional[torch.Tensor] = None   # int32 [n_seqs] view, for parts written in Python
     pos0_dev: Optional[torch.Tensor] = None
     cu_q_dev: Optional[torch.Tensor] = None
@@ -234,6 +235,12 @@ class PositionEncoding(Part):
         attention), else None (the default): the mixer then calls `encode`."""
         return None
 
+    def scaled_rotary_constants(self):
+        """(inv_freq, rotary_dim, pairing, factor on cosine and sine) for mixers whose kernels apply a rotation
+        that also scales; the default: what `rotary_constants` says, with factor 1."""
+        rot = self.rotary_constants()
+        return None if rot is None else (*rot, 1.0)
+
 
 class Mixer(Part):
     def cache_request(self) -> CacheRequest:
@@ -286,7 +293,19 @@ class StepInput(Part):
     (int32 on the device, padding included) and the embedded rows `x` (fp32 [tokens, hidden]).  It may
     change `x` in place (a norm or a bias on the embedding) and may publish tensors for the blocks in
     `ctx.shared[name]` (an input that every layer reads, computed from the ids once).  Its tensors are
-    found under the prefix that `ModelSpec.inputs` names beside its spec."""
+    found under the prefix that `ModelSpec.inputs` names beside its spec.
+
+    An input may keep state per sequence like a mixer: what `cache_request` asks for is in `ctx.input_view` while it
+    runs.  The first input of a model may take the embedding over (`embeds` True): the model then calls
+    `embed(table, tokens, x, scale, ctx)`, which writes the embedded rows with the input's own change in one pass, and
+    does not call its `prepare`."""
+    embeds = False
+
+    def cache_request(self) -> CacheRequest:
+        return None
+
+    def embed(self, table, tokens, x, scale: float, ctx: StepContext) -> None:
+        raise NotImplementedError
 
     def prepare(self, tokens, x, ctx: StepContext) -> None:
         raise NotImplementedError

@@ -1,4 +1,5 @@
-"""Arrangement of a layer's parts.  "shared_norm": h = norm1(x); x += mixer(h) + ffn(h) (one norm, read by both
+"""Arrangement of a layer's parts.  "two_norms": x += mixer(norm1(x)) + ffn(norm2(x)), both norms of the same
+x.  "shared_norm": h = norm1(x); x += mixer(h) + ffn(h) (one norm, read by both
 sublayers).  "prenorm": x += mixer(norm1(x)); x += ffn(norm2(x)) (the second
 half left out for a layer without a feed-forward)
 (src/layers/block.rs:19-24,63-65; the residual uses the un-normed input,
@@ -197,7 +198,45 @@ class SharedNormBlock(Block):
         ctx.norm_ahead = None
 
 
+class TwoNormsBlock(Block):
+    """Both sublayers read the same residual, each through a norm of its own:
+
+        x <- x + (mixer(norm1(x)) + ffn(norm2(x)))             (the second term left out for a layer without a feed-forward)
+
+    The norms run first, in one pass over the rows where their kind can (`forward_pair`); then both sublayers add into the
+    fp32 residual, which neither reads."""
+    graph_safe = True
+
+    def __init__(self, layer_spec, norm1, mixer, norm2, ffn, rt: Runtime):
+        if ffn is not None and norm2 is None:
+            raise ValueError("block 'two_norms' with a feed-forward needs a second norm (LayerSpec.ffn_norm_name)")
+        self.norm1, self.mixer, self.norm2, self.ffn, self.rt = norm1, mixer, norm2, ffn, rt
+
+    def forward(self, x, ctx: StepContext, cache_view, writes_cache: bool) -> None:
+        ctx.rows_ahead = None
+        ws, T = self.rt.workspace, ctx.n_tokens
+        h = ws.take("block.normed", x.shape, self.rt.dtype)
+        h2 = None
+        if self.ffn is not None:
+            h2 = ws.take("block.normed2", x.shape, self.rt.dtype)
+            pair = getattr(self.norm1, "forward_pair", None)
+            if pair is None or not pair(self.norm2, x, h, h2, ctx, T):
+                self.norm1.forward(x, h, ctx, rows=T)
+                self.norm2.forward(x, h2, ctx, rows=T)
+        else:
+            self.norm1.forward(x, h, ctx, rows=T)
+        # only the block's last addition may write the next block's norm ahead: the rows are final then
+        ahead = first_norm_request_of(ctx.next_block, ctx)
+        ctx.norm_ahead = ahead if self.ffn is None else None
+        self.mixer.forward(h, x, ctx, cache_view, writes_cache)
+        if self.ffn is not None:
+            ctx.norm_ahead = ahead
+            self.ffn.forward(h2, x, ctx)
+        ctx.norm_ahead = None
+
+
 register_part("block", "prenorm", PreNormBlock)
+register_part("block", "two_norms", TwoNormsBlock)
 register_part("block", "shared_norm", SharedNormBlock)
 register_part("block", "outnorm", OutputNormBlock)
 register_part("block", "hyper", HyperConnectionBlock)

@@ -1,15 +1,23 @@
 """Grouped-query attention with biases on the input projections, a weighted RMS norm on every head of q and of k,
-a value size that may differ from the query/key size, and a sigmoid gate on the concatenated heads:
+a value size that may differ from the query/key size, values mixed with another layer's, and a sigmoid gate on the
+concatenated heads or on each head:
 
     q = W_q h + b_q,  k = W_k h + b_k,  v = W_v h + b_v                       (`bias`: the b's exist)
     q_head <- q_head / rms(q_head) * w_q,  k likewise with w_k                (`qk_norm` "head": weights of length
                                                                                head_dim, the same for all heads; before
                                                                                the rotation)
-    rotation by the mixer's position part (a plain rotary encoding, either pairing, any number of rotated dimensions)
-    a = softmax(q . k * scale over the visible keys) v                        (causal, optionally a sliding `window`)
-    y = W_o (a * sigmoid(W_g h))                                              (`gate`: W_g exists)
+    rotation by the mixer's position part (a rotary encoding, either pairing, any number of rotated dimensions, cosine and
+                                                                               sine times a factor)
+    v <- (1 - lambda) v + lambda v_first                                      (`v_mix` "mix": v_first are the values, as
+                                                                               projected, of the layer with `v_mix` "source",
+                                                                               for the same token; the mixed v is cached)
+    a = softmax(q . k * scale over the visible keys) v                        (causal, optionally a sliding `window` behind
+                                                                               which the first `keep` positions stay visible)
+    y = W_o (a * sigmoid(W_g h))                                              (`gate` True: a gate per number; "head": one
+                                                                               per head, the same for all its numbers)
 
-Tensors: q, k, v (+ q.b, k.b, v.b), q.norm, k.norm, g, o.  One product makes [q | k | v | g] in fp32; one kernel adds
+Tensors: q, k, v (+ q.b, k.b, v.b), q.norm, k.norm, vmix (one number; the source layer has it too and does not use it),
+g, o.  One product makes [q | k | v | g] in fp32; one kernel adds
 the biases, norms, rotates, rounds once and writes the packed row and the cache; the library's attention kernels run
 on heads padded with zeros to one common size D >= max(head_dim, v_dim) (a multiple of 16 for the tensor-core kernels),
 so that keys and values share the paged cache's geometry; one kernel drops the padding and applies the gate; W_o adds
@@ -42,7 +50,15 @@ class GatedAttention(Mixer):
         self.scale = float(spec["scale"])
         self.eps = float(spec.get("eps", 0.0))
         self.has_bias = bool(spec.get("bias", False))
-        self.has_gate = bool(spec.get("gate", False))
+        self.gate = spec.get("gate", False)
+        if self.gate not in (False, True, None, "head"):
+            raise ValueError(f"gate must be true, false or 'head', got {self.gate!r}")
+        self.has_gate = bool(self.gate)
+        self.keep = int(spec.get("keep") or 0)
+        self.v_mix = spec.get("v_mix")
+        if self.v_mix not in (None, "source", "mix"):
+            raise ValueError(f"v_mix must be 'source', 'mix' or None, got {self.v_mix!r}")
+        self.lam = 0.0
         qk_norm = spec.get("qk_norm")
         if qk_norm not in (None, "head"):
             raise ValueError(f"qk_norm must be 'head' or None, got {qk_norm!r}")
@@ -54,10 +70,10 @@ class GatedAttention(Mixer):
         self.head_dim = -(-widest // 16) * 16 if rt.fast else widest
         pos = spec["position"]
         self.position = part_class("position", pos.kind)(pos, self.qk_dim, rt)
-        rot = getattr(self.position, "rotary_constants", lambda: None)()
+        rot = getattr(self.position, "scaled_rotary_constants", lambda: None)()
         if rot is None:
             raise ValueError("gated attention takes a rotary position part")
-        self.inv_freq, self.rotary_dim, self.pairing = rot
+        self.inv_freq, self.rotary_dim, self.pairing, self.rot_mul = rot
         self.q_dim = self.heads * self.qk_dim
         self.k_dim = self.kv_heads * self.qk_dim
         self.kv_v_dim = self.kv_heads * self.v_dim
@@ -74,13 +90,20 @@ class GatedAttention(Mixer):
             specs["q.norm"] = TensorSpec((self.qk_dim,), "ones_plus_normal")
             specs["k.norm"] = TensorSpec((self.qk_dim,), "ones_plus_normal")
         if self.has_gate:
-            specs["g"] = TensorSpec((self.a_dim, h))
+            specs["g"] = TensorSpec((self.heads if self.gate == "head" else self.a_dim, h))
+        if self.v_mix:
+            specs["vmix"] = TensorSpec(())
         return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         dt = self.rt.dtype
         rows = [tensors["q"].to(dt), tensors["k"].to(dt), tensors["v"].to(dt)] + ([tensors["g"].to(dt)] if self.has_gate else [])
+        n = sum(r.shape[0] for r in rows)
+        if n % 8:                                 # the tensor-core projection wants output rows of whole 16 bytes
+            rows.append(torch.zeros((8 - n % 8, rows[0].shape[1]), dtype=dt, device=rows[0].device))
         self.proj = Linear(torch.cat(rows, dim=0), self.rt)
+        if self.v_mix == "mix":
+            self.lam = float(tensors["vmix"])
         self.o = Linear(tensors["o"], self.rt)
         if self.has_bias:
             self.bias = torch.cat([tensors[n].to(torch.float32) for n in ("q.b", "k.b", "v.b")]).contiguous()
@@ -89,30 +112,35 @@ class GatedAttention(Mixer):
             self.wk = tensors["k.norm"].to(torch.float32).contiguous()
 
     def cache_request(self) -> KVRequest:
-        return KVRequest(self.kv_heads, self.head_dim, self.window)
+        return KVRequest(self.kv_heads, self.head_dim, self.window, keep=self.keep)
 
     def weight_bytes(self) -> int:
         return self.proj.nbytes() + self.o.nbytes()
 
     def cut_by_length_key(self):
-        return ("gated_attention", self.heads, self.kv_heads, self.head_dim, self.window, self.rt.fast)
+        return ("gated_attention", self.heads, self.kv_heads, self.head_dim, self.window, self.keep, self.rt.fast)
 
     def cut_by_length(self, pos0, cache_view) -> bool:
         if not self.rt.fast or cache_view is None:
             return False
         from . import fast_attention
         return fast_attention.wants_length_cut(pos0, self.kv_heads, self.heads // self.kv_heads, self.window,
-                                               cache_view.group.page_tokens, self.head_dim)
+                                               cache_view.group.page_tokens, self.head_dim, keep=self.keep)
 
     def forward(self, xn, residual, ctx: StepContext, cache_view, writes_cache: bool) -> None:
         rt, ws, T, D = self.rt, self.rt.workspace, ctx.n_tokens, self.head_dim
         kv = cache_view.struct
         n_qkv = self.q_dim + self.k_dim + self.kv_v_dim
-        proj = ws.take("gattn.proj", (T, self.proj.out_features), torch.float32)
+        # the source layer's projection stays as it is until the step's last mixing layer has read its values
+        proj = ws.take("gattn.proj_source" if self.v_mix == "source" else "gattn.proj", (T, self.proj.out_features), torch.float32)
         self.proj.apply(xn, proj, T, ctx.stream)
+        if self.v_mix == "source":
+            ctx.shared["v_first"] = proj[:, self.q_dim + self.k_dim:n_qkv]
+        v_first = ctx.shared["v_first"] if self.v_mix == "mix" else None
         qkv = ws.take("attn.qkv", (T, (self.heads + 2 * self.kv_heads) * D), rt.dtype)
         B.qkv_prep(proj, self.bias, qkv, ctx.batch, kv, self.heads, self.qk_dim, self.v_dim, self.inv_freq, self.rotary_dim,
-                   self.pairing, self.wq, self.wk, self.eps, writes_cache, rt.err, ctx.stream)
+                   self.pairing, self.wq, self.wk, self.eps, writes_cache, rt.err, ctx.stream, rot_mul=self.rot_mul,
+                   v_first=v_first, lam=self.lam)
         out = ws.take("attn.out", (T, self.heads * D), rt.dtype)
         from_cache = ctx.kind == "decode" or not writes_cache
         if from_cache and ctx.kind == "prompt":
@@ -128,7 +156,8 @@ class GatedAttention(Mixer):
             B.attention_plain(qkv, out, ctx.batch, kv, self.heads, self.scale, from_cache, rt.err, ctx.stream)
         if self.has_gate or D != self.v_dim:
             gated = ws.take("gattn.gated", (T, self.a_dim), rt.dtype)
-            B.gate_mul(out, proj[:, n_qkv:] if self.has_gate else None, gated, T, self.heads, D, self.v_dim, ctx.stream)
+            B.gate_mul(out, proj[:, n_qkv:] if self.has_gate else None, gated, T, self.heads, D, self.v_dim, ctx.stream,
+                       per_head=self.gate == "head")
             out = gated
         self.o.apply(out, residual, T, ctx.stream, add_residual=True, ctx=ctx)
 

@@ -98,8 +98,19 @@ class LayerNorm(Norm):
 
     def forward(self, x, out, ctx, rows_idx=None, rows=None) -> None:
         n = rows if rows is not None else (rows_idx.numel() if rows_idx is not None else x.shape[0])
-        B.streams_norm(x, 1, self.hidden_size, n, ctx.stream, w=self.weight, b=self.bias, eps=self.eps, out=out,
-                       rows_idx=rows_idx)
+        if out.data_ptr() == x.data_ptr():               # in place: the kernel of the streams reads a row whole first
+            B.streams_norm(x, 1, self.hidden_size, n, ctx.stream, w=self.weight, b=self.bias, eps=self.eps, out=out,
+                           rows_idx=rows_idx)
+        else:
+            B.layernorm(x, out, self.weight, self.bias, self.eps, n, ctx.stream, rows_idx=rows_idx)
+
+    def forward_pair(self, other, x, out, other_out, ctx, rows: int) -> bool:
+        """This norm and `other` of the same rows in one pass, if `other` is of this kind with the same constant
+        (they share mean and variance); False: nothing was launched."""
+        if not isinstance(other, LayerNorm) or other.eps != self.eps or other.hidden_size != self.hidden_size:
+            return False
+        B.layernorm(x, out, self.weight, self.bias, self.eps, rows, ctx.stream, second=(other.weight, other.bias, other_out))
+        return True
 
     def forward_streams(self, xs, n_streams: int, out, ctx, rows: int, rows_idx=None, in_coef=None, update=None,
                         clear=None) -> None:
