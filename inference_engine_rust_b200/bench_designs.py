@@ -20,7 +20,7 @@ LAUNCHERS = ["embed_gather", "rmsnorm", "rope_kv_store", "silu_mul", "gemm_plain
              "mlstm_recur", "gated_head_norm", "latent_norm_store", "latent_attention_prompt", "latent_attention_decode_tc",
              "latent_attention_decode", "router_topk", "moe_scale", "add_normed", "cast_rows", "scale_values", "qk_prep",
              "rglru_conv", "rglru_gates", "rglru_scan", "qkv_prep", "gate_mul", "router_grouped", "gated_act_mul",
-             "token_shift", "wkv_decay", "wkv_recur", "wkv_finish", "latent_prep", "head_gate_mul"]
+             "token_shift", "wkv_decay", "wkv_recur", "wkv_finish", "latent_prep", "head_gate_mul", "layernorm", "embed_pairs"]
 GEMMS = {"gemm_plain", "gemm_tc", "gemm_rows", "gemm_tc_scaled", "gemm_tc_gated", "gemm_tc_gated_scaled"}
 
 
@@ -56,6 +56,8 @@ class KernelClock:
                     nbytes = w.numel() * w.element_size() + M * K * x.element_size() + M * N * o.element_size()
                 elif _name == "attention_prefill":
                     label = f"{_name} [head {args[5]}]"           # a model may run it at more than one head size
+                elif _name == "latent_prep":
+                    label = f"{_name} [{' '.join(n for n in ('q', 'down', 'dq') if kw.get(n) is not None)}]"
                 if out is not False:
                     self.records.append((label, a, b, flops, nbytes))
                 return out
@@ -189,7 +191,7 @@ def _costs(cfg: dict, T: int, n_seqs: int, ctx: int, prompt: bool) -> Dict[str, 
             wide = m["kv_rank"] + m["rot_dim"]
             row = m["heads"] * (m["dim"] + m["rot_dim"]) + wide + m["heads"]
             out[f"attention_prefill [head {P}]"] = (4.0 * m["heads"] * P * T * (T + 1) / 2, True, T * 4 * m["heads"] * P * 2)
-            out["latent_prep"] = (0.0, False, T * (row * 4 + wide * 4 + m["heads"] * P * 2))
+            out["latent_prep"] = (0.0, False, T * (row * 4 + wide * 4 + (m["heads"] * P * 2 if prompt else 0)))
             out["head_gate_mul"] = (0.0, False, T * m["heads"] * (P + m["vdim"]) * 2)
             out["latent_attention_decode"] = out["latent_attention_decode_tc"] = (
                 2.0 * n_seqs * m["heads"] * ctx * (wide + m["kv_rank"]), True,
@@ -199,6 +201,42 @@ def _costs(cfg: dict, T: int, n_seqs: int, ctx: int, prompt: bool) -> Dict[str, 
             r = mlp["router"]
             out["moe_scale"] = (0.0, False, T * r["experts"] * mlp["expert"]["ff"] * 4)
             out["router_grouped"] = (0.0, False, T * r["experts"] * 8)
+    elif cfg.get("architecture") == "Botulorn":
+        H = cfg["width"]
+        out["embed_pairs"] = (0.0, False, T * H * 8)
+        out["layernorm"] = (0.0, False, T * H * 8)                      # one read of the row, two normed rows
+        by = {l["type"]: l["mixer"] for l in cfg["layers"]}
+
+        def seen_by(T, W, keep):
+            """(query, key) pairs of a prompt under a window of W behind which `keep` first positions stay visible."""
+            return sum(min(i + 1, W + min(keep, max(i + 1 - W, 0))) for i in range(T))
+        if "attention" in by:
+            m = by["attention"]
+            mask = m.get("mask") or {}
+            W, keep = mask.get("size") or (1 << 30), mask.get("keep_first") or 0
+            D = -(-max(m["dim"], m["vdim"]) // 16) * 16
+            qd, kd, vd, ad = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
+            packed = (m["heads"] + 2 * m["kv_heads"]) * D
+            out["qkv_prep"] = (0.0, False, T * ((qd + kd + vd) * 4 + packed * 2 + 2 * m["kv_heads"] * D * 2))
+            out["gate_mul"] = (0.0, False, T * (m["heads"] * D * 2 + m["heads"] * 4 + ad * 2))
+            if prompt:
+                out[f"attention_prefill [head {D}]"] = (4.0 * m["heads"] * D * seen_by(T, W, keep), True,
+                                                        T * (2 * m["heads"] * D + 2 * m["kv_heads"] * D) * 2)
+            out["attention_decode_tc"] = (0.0, False, n_seqs * min(ctx, W + keep) * 2 * m["kv_heads"] * D * 2)
+        if "latent_attention" in by:
+            m = by["latent_attention"]
+            W = (m.get("mask") or {}).get("size") or (1 << 30)
+            P = -(-max(m["dim"] + m["rot_dim"], m["vdim"]) // 16) * 16
+            wide, hq = m["kv_rank"] + m["rot_dim"], m["heads"] * (m["dim"] + m["rot_dim"])
+            if prompt:
+                out[f"attention_prefill [head {P}]"] = (4.0 * m["heads"] * P * seen_by(T, W, 0), True, T * 4 * m["heads"] * P * 2)
+            out["latent_prep [q]"] = (0.0, False, T * (hq * 4 + m["heads"] * P * 2))
+            out["latent_prep [down dq]"] = (0.0, False, T * ((wide + m["q_rank"]) * 4 + wide * 4 + m["q_rank"] * 2))
+            out["head_gate_mul"] = (0.0, False, T * m["heads"] * (P + m["vdim"]) * 2)
+            seen = min(ctx, W)
+            out["latent_attention_decode"] = out["latent_attention_decode_tc"] = (
+                2.0 * n_seqs * m["heads"] * seen * (wide + m["kv_rank"]), True,
+                n_seqs * seen * wide * 2 + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"] * 2)
     else:
         hd = cfg["num_attention_heads"] * cfg["head_dim"]
         kvd = cfg["num_key_value_heads"] * cfg["head_dim"]
