@@ -159,15 +159,15 @@ def _botulorn(width, vocab, layers, heads, kv_heads, dim, vdim, window, keep, la
         kind, mixer = mixers[0 if i % 4 in (0, 3) else 1]
         out.append({"type": kind, "mixer": copy.deepcopy(mixer), "mlp": {"kind": "dense", "ff": ff}})
     return {"architecture": "Botulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
-            "embedding": {"scale": 8.0, "bigram": {"buckets": buckets, "mul_prev": 1009, "mul_cur": 31}}, "layers": out}
+            "embedding": {"scale": 8.0, "bigram": {"buckets": buckets, "mul_prev": 1009, "mul_cur": 131}}, "layers": out}
 
 
 # Botulorn at the width, head count, head size and feed-forward size of Mistral 7B (latent attention with 128 unrotated and 64
-# rotated numbers per head over latents of 1,536 and 512; windows of 4,096 positions, the first four kept), and a tiny one that
+# rotated numbers per head over latents of 1,536 and 512; windows of 4,096 positions, the first eight kept), and a tiny one that
 # runs anywhere in seconds.
-PRESETS["botulorn-7b-sizes"] = _botulorn(4096, 32000, 32, 32, 8, 128, 128, 4096, 4, 128, 64, 128, 1536, 512, 4096, 14336, 65521, 4096)
+PRESETS["botulorn-7b-sizes"] = _botulorn(4096, 32000, 32, 32, 8, 128, 128, 4096, 8, 128, 64, 128, 1536, 512, 4096, 14336, 65521, 4096)
 # the same at the sizes of Mistral NeMo 12B (width 5,120, a vocabulary of 131,072)
-PRESETS["botulorn-12b-sizes"] = _botulorn(5120, 131072, 40, 32, 8, 128, 128, 4096, 4, 128, 64, 128, 1536, 512, 4096, 14336, 65521, 4096)
+PRESETS["botulorn-12b-sizes"] = _botulorn(5120, 131072, 40, 32, 8, 128, 128, 4096, 8, 128, 64, 128, 1536, 512, 4096, 14336, 65521, 4096)
 PRESETS["botulorn-tiny"] = _botulorn(80, 320, 4, 6, 3, 16, 24, 20, 2, 12, 8, 16, 24, 40, 28, 72, 101, 64)
 
 

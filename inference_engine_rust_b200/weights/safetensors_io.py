@@ -195,4 +195,4 @@ def write_safetensors(path: str, tensors: Mapping[str, torch.Tensor],
         f.write(blob)
         for name in order:
             t = tensors[name].detach().cpu().contiguous()
-            f.write(t.view(torch.uint8).reshape(-1).numpy().tobytes() if t.numel() else b"")
+            f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")
