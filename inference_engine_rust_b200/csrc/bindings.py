@@ -150,7 +150,7 @@ def _declare(lib) -> None:
         "iert_token_shift": [P, c_int, LL, P, LL, LL, P, c_int, c_int, P, POINTER(BatchView), S],
         "iert_wkv_decay": [P, LL, c_int, P, P, c_int, P, P, c_int, LL, c_int, P, LL, LL, POINTER(BatchView), S],
         "iert_wkv_finish": [P, P, LL, P, c_float, c_float, P, c_int, POINTER(BatchView), c_int, c_int, S],
-        "iert_latent_decode_tc_plan": [c_int, c_int, c_int, POINTER(c_int), POINTER(c_int)],
+        "iert_latent_decode_tc_plan": [c_int, c_int, c_int, c_int, c_int, POINTER(c_int), POINTER(c_int)],
         "iert_router_topk": [P, LL, P, c_int, c_int, c_int, P, P, P, S],
         "iert_moe_scale": [P, c_int, LL, P, c_int, c_int, c_int, P, P, LL, P, c_int, S],
         "iert_router_grouped": [P, LL, LL, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
@@ -770,17 +770,19 @@ def head_gate_mul(attn, head: int, out, V: int, H: int, gate, batch: BatchView, 
                                     stream), "head_gate_mul")
 
 
-def latent_decode_tc_plan(n_seqs: int, H: int, table_width: int):
-    """(heads padded to whole MMA tiles, runs a sequence is cut into) of the tensor-core one-token kernel."""
+def latent_decode_tc_plan(n_seqs: int, H: int, rank: int, rot_dim: int, table_width: int):
+    """(heads padded to whole MMA tiles, runs a sequence is cut into) of the tensor-core one-token kernel; `table_width`:
+    pages of the longest walk."""
     hpad, splits = c_int(0), c_int(0)
-    core().iert_latent_decode_tc_plan(n_seqs, H, table_width, byref(hpad), byref(splits))
+    core().iert_latent_decode_tc_plan(n_seqs, H, rank, rot_dim, table_width, byref(hpad), byref(splits))
     return hpad.value, splits.value
 
 
 def latent_attention_decode_tc(q, w_uk, w_uv, out, batch: BatchView, kv: KvView, H: int, D: int, V: int, scale: float, sink,
                                hpad: int, splits: int, qa, part_m, part_l, part_acc, err, stream, rot_dim: int = 0,
                                gate=None, inv_freq=None, rot_mul: float = 1.0, pairing: int = PAIR_HALF) -> bool:
-    """One-token latent attention on the tensor cores (bf16, rank a multiple of 32 up to 512, pages of 64):
+    """One-token latent attention on the tensor cores (bf16, rank a multiple of 8 up to 512, pages of 64; tcgen05, or mma.sync
+    where ranks and rotated parts in whole MMA steps ask for it or IERT_LATENT_UMMA=0 does):
     the absorbed queries, the split attention over the cached latents, the merge with the sink and W_uv.  `q`: bf16 with its
     rotated part turned already, or the fp32 projection, whose rotated part is turned here by `inv_freq`, `rot_mul`, `pairing`.
     Returns False, having launched nothing, for sizes it does not take."""

@@ -5,7 +5,7 @@
 //   S = Qa C^T   ([heads x rank] x [rank x keys]),   P = softmax with a sink,   L = P C  ([heads x keys] x [keys x rank])
 //
 // which is multi-query attention whose keys and values are the same rows.  W_uv is applied to L at the
-// end, once per head.  Three kernels:
+// end, once per head.  Three kernels (the one in the middle is the one of latent_decode_umma.cu where that takes the sizes):
 //   latent_absorb_q       qa [T, Hpad, rank] bf16 from q and W_uk (rows of padding heads are zero); q either in bf16 with
 //                         its rotated part turned already, or the fp32 projection itself, turned on the way
 //   latent_decode_tc      a CTA takes (sequence, a run of 64-key tiles, up to 32 heads): the tile of C comes
@@ -16,9 +16,11 @@
 //   latent_decode_merge   merges the runs in order, adds the sink's term exp(sink - M) to the denominator,
 //                         and multiplies by W_uv: out [T, H*V].
 // A window, a chunk or kept first positions of the cache view choose which pages are walked and which rows count.
-// Sizes: rank a multiple of 32 up to 512, pages of 64 positions, a bf16 cache.  Anything else is refused
+// Sizes: rank a multiple of 32 (of 8 for the kernel of latent_decode_umma.cu) up to 512, pages of 64 positions, a bf16 cache.  Anything else is refused
 // (IERT_BAD_ARGUMENT) and the caller runs the plain kernel.
 #include "common.cuh"
+
+#include <cstdlib>
 
 using namespace iert;
 
@@ -37,69 +39,87 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ uint32_t lds32(const __nv_bfloat16* p) { return *reinterpret_cast<const uint32_t*>(p); }
 
-// qa[t, h, :] = sum_d q[t, h, d] W_uk[h*D + d, :].  A block of 256 threads takes one (token, head): 64 threads
-// across the rank (eight columns each, 16-byte loads of the weights) times four groups along d, added
-// through shared memory in a fixed order.
+// qa[t, h, :] = sum_d q[t, h, d] W_uk[h*D + d, :].  A block of 256 threads takes one head of TT tokens, so that the
+// head's weights are read once for all of them: 64 threads across the rank (eight columns each, 16-byte loads of the
+// weights) times four groups along d, added through shared memory in a fixed order.
 constexpr int ABSORB_THREADS = 256;
 
 // TQ float: q is the projection as it stands, and the R last numbers of a head are turned here (inv_freq, rot_mul, pairing).
-template <typename TQ>
+template <typename TQ, int TT>
 __global__ void __launch_bounds__(ABSORB_THREADS)
 latent_absorb_q_kernel(const TQ* __restrict__ q, long long ldq, const __nv_bfloat16* __restrict__ w_uk,
                        __nv_bfloat16* __restrict__ qa, int H, int Hpad, int D, int R, int rank, const float* __restrict__ inv_freq,
                        float rot_mul, int pairing, IertBatchView b) {
   extern __shared__ float sm_q[];
-  float* q_s = sm_q;                    // [D]
-  float* part = sm_q + D;               // [4][rank]
+  float* q_s = sm_q;                    // [TT][D]
+  float* part = sm_q + TT * D;          // [4][TT][rank]
   pdl_launch_dependents();
+  const int t0 = blockIdx.x * TT, h = blockIdx.y, n_t = min(TT, b.n_tokens - t0);
   pdl_wait();
-  const int t = blockIdx.x, h = blockIdx.y;
-  __nv_bfloat16* dst = qa + ((size_t)t * Hpad + h) * (rank + R);
-  if (h >= H) {
-    for (int r = threadIdx.x; r < rank + R; r += blockDim.x) dst[r] = __float2bfloat16_rn(0.f);
+  if (h >= H) {                         // heads that only fill the MMA tile
+    for (int i = threadIdx.x; i < n_t * (rank + R); i += blockDim.x)
+      qa[((size_t)(t0 + i / (rank + R)) * Hpad + h) * (rank + R) + i % (rank + R)] = __float2bfloat16_rn(0.f);
     return;
   }
-  const TQ* qh = q + (size_t)t * ldq + (size_t)h * (D + R);
-  for (int d = threadIdx.x; d < D; d += blockDim.x) q_s[d] = to_f32(qh[d]);
+  for (int i = threadIdx.x; i < TT * D; i += blockDim.x) {
+    const int t = i / D, d = i - t * D;
+    q_s[i] = t < n_t ? to_f32(q[(size_t)(t0 + t) * ldq + (size_t)h * (D + R) + d]) : 0.f;
+  }
   if (sizeof(TQ) == 4) {                // one token per sequence: token t is sequence t's
-    const int half = R / 2, pos = b.pos0[t];
-    for (int k = threadIdx.x; k < half; k += blockDim.x) {
+    const int half = R / 2;
+    for (int i = threadIdx.x; i < n_t * half; i += blockDim.x) {
+      const int t = t0 + i / half, k = i % half, pos = b.pos0[t];
+      const TQ* v = q + (size_t)t * ldq + (size_t)h * (D + R) + D;
+      __nv_bfloat16* dst = qa + ((size_t)t * Hpad + h) * (rank + R) + rank;
       const int i0 = pairing == IERT_PAIR_INTERLEAVED ? 2 * k : k, i1 = pairing == IERT_PAIR_INTERLEAVED ? 2 * k + 1 : k + half;
-      const float u = to_f32(qh[D + i0]), v = to_f32(qh[D + i1]);
+      const float x = to_f32(v[i0]), y = to_f32(v[i1]);
       float sn, co;
       sincosf((float)pos * inv_freq[k], &sn, &co);
       sn *= rot_mul;
       co *= rot_mul;
-      dst[rank + i0] = __float2bfloat16_rn(u * co - v * sn);
-      dst[rank + i1] = __float2bfloat16_rn(v * co + u * sn);
+      dst[i0] = __float2bfloat16_rn(x * co - y * sn);
+      dst[i1] = __float2bfloat16_rn(y * co + x * sn);
     }
   } else {
-    for (int i = threadIdx.x; i < R; i += blockDim.x) dst[rank + i] = __float2bfloat16_rn(to_f32(qh[D + i]));   // turned already
+    for (int i = threadIdx.x; i < n_t * R; i += blockDim.x) {                        // turned already
+      const int t = t0 + i / R, k = i % R;
+      qa[((size_t)t * Hpad + h) * (rank + R) + rank + k] = __float2bfloat16_rn(to_f32(q[(size_t)t * ldq + (size_t)h * (D + R) + D + k]));
+    }
   }
   __syncthreads();
   const int grp = threadIdx.x >> 6, lane64 = threadIdx.x & 63;
   const int d_lo = grp * ((D + 3) / 4), d_hi = min(D, d_lo + (D + 3) / 4);
   for (int r0 = lane64 * 8; r0 < rank; r0 += 64 * 8) {
-    float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    float a[TT][8];
+#pragma unroll
+    for (int t = 0; t < TT; ++t)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[t][e] = 0.f;
     const __nv_bfloat16* w = w_uk + (size_t)h * D * rank + r0;
-#pragma unroll 4
+#pragma unroll 8
     for (int d = d_lo; d < d_hi; ++d) {
       const uint4 v = *reinterpret_cast<const uint4*>(w + (size_t)d * rank);
       const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&v);
-      const float qd = q_s[d];
+      float f[8];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(p[e]);
-        a[2 * e] = fmaf(qd, f.x, a[2 * e]);
-        a[2 * e + 1] = fmaf(qd, f.y, a[2 * e + 1]);
+      for (int e = 0; e < 4; ++e) { const float2 two = __bfloat1622float2(p[e]); f[2 * e] = two.x; f[2 * e + 1] = two.y; }
+#pragma unroll
+      for (int t = 0; t < TT; ++t) {
+        const float qd = q_s[t * D + d];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[t][e] = fmaf(qd, f[e], a[t][e]);
       }
     }
 #pragma unroll
-    for (int e = 0; e < 8; ++e) part[grp * rank + r0 + e] = a[e];
+    for (int t = 0; t < TT; ++t)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) part[(grp * TT + t) * rank + r0 + e] = a[t][e];
   }
   __syncthreads();
-  for (int r = threadIdx.x; r < rank; r += blockDim.x)
-    dst[r] = __float2bfloat16_rn((part[r] + part[rank + r]) + (part[2 * rank + r] + part[3 * rank + r]));
+  const int all = TT * rank;
+  for (int i = threadIdx.x; i < n_t * rank; i += blockDim.x)
+    qa[((size_t)(t0 + i / rank) * Hpad + h) * (rank + R) + i % rank] =
+        __float2bfloat16_rn((part[i] + part[all + i]) + (part[2 * all + i] + part[3 * all + i]));
 }
 
 template <int MT>
@@ -286,32 +306,30 @@ latent_decode_tc_kernel(const __nv_bfloat16* __restrict__ qa, IertBatchView b, I
 
 constexpr int MERGE_THREADS = 256;
 
-template <typename T>
+// A block merges the runs of one head of TT sequences and multiplies each by the head's W_uv, whose rows are read once for
+// all of them.
+template <typename T, int TT>
 __global__ void __launch_bounds__(MERGE_THREADS)
 latent_decode_merge_kernel(const float* __restrict__ part_m, const float* __restrict__ part_l,
                            const float* __restrict__ part_acc, int splits, int Hpad, int rank,
                            const float* __restrict__ sink, const float* __restrict__ gate, const T* __restrict__ w_uv,
                            T* __restrict__ out, IertBatchView b, int H, int V) {
   extern __shared__ float sm[];
-  float* lat = sm;                 // [rank]
-  float* wgt = sm + rank;          // [64]
+  float* lat = sm;                 // [TT][rank]
+  float* wgt = sm + TT * rank;     // [TT][64]
   pdl_launch_dependents();
+  const int t0 = blockIdx.x * TT, h = blockIdx.y, n_t = min(TT, b.n_seqs - t0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
-  const int t = blockIdx.x, h = blockIdx.y;
-  T* o = out + ((size_t)t * H + h) * V;
-  if (b.slot_ids[t] < 0) {
-    for (int e = threadIdx.x; e < V; e += MERGE_THREADS) o[e] = from_f32<T>(0.f);
-    return;
-  }
-  if (threadIdx.x < 32) {                 // splits <= 64: two runs per lane
-    const int lane = threadIdx.x;
+  for (int t = warp; t < TT; t += MERGE_THREADS / 32) {          // splits <= 64: two runs per lane
+    const bool live = t < n_t && b.slot_ids[t0 + t] >= 0;        // a padding sequence: weights of zero
     float mi[2], li[2];
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
       const int i = lane + 32 * k;
-      const size_t row = ((size_t)t * splits + (i < splits ? i : 0)) * Hpad + h;
-      mi[k] = i < splits ? part_m[row] : -INFINITY;
-      li[k] = i < splits ? part_l[row] : 0.f;
+      const size_t row = ((size_t)(live ? t0 + t : 0) * splits + (i < splits ? i : 0)) * Hpad + h;
+      mi[k] = live && i < splits ? part_m[row] : -INFINITY;
+      li[k] = live && i < splits ? part_l[row] : 0.f;
     }
     const float snk = sink ? sink[h] : -INFINITY;
     const float M = fmaxf(warp_max(fmaxf(mi[0], mi[1])), snk);
@@ -324,50 +342,65 @@ latent_decode_merge_kernel(const float* __restrict__ part_m, const float* __rest
     const float L = warp_sum(part) + (sink ? expf(snk - M) : 0.f);
     const float inv = L > 0.f ? 1.0f / L : 0.f;
 #pragma unroll
-    for (int k = 0; k < 2; ++k) wgt[lane + 32 * k] = lane + 32 * k < splits ? w[k] * inv : 0.f;
+    for (int k = 0; k < 2; ++k) wgt[t * 64 + lane + 32 * k] = lane + 32 * k < splits ? w[k] * inv : 0.f;
   }
   __syncthreads();
   // the runs' partial sums, eight loads in flight per thread; an empty run's row (weight 0) is never read
-  for (int r = threadIdx.x; r < rank; r += MERGE_THREADS) {
+  for (int j = threadIdx.x; j < TT * rank; j += MERGE_THREADS) {
+    const int t = j / rank, r = j - t * rank;
+    const float* wt = wgt + t * 64;
     float a = 0.f;
     for (int i0 = 0; i0 < splits; i0 += 8) {
       float v[8];
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
         const int i = i0 + k;
-        v[k] = (i < splits && wgt[i] != 0.f) ? part_acc[(((size_t)t * splits + i) * Hpad + h) * rank + r] : 0.f;
+        v[k] = (i < splits && wt[i] != 0.f) ? part_acc[(((size_t)(t0 + t) * splits + i) * Hpad + h) * rank + r] : 0.f;
       }
 #pragma unroll
-      for (int k = 0; k < 8; ++k) a = fmaf(wgt[(i0 + k) & 63], v[k], a);
+      for (int k = 0; k < 8; ++k) a = fmaf(wt[(i0 + k) & 63], v[k], a);
     }
-    lat[r] = a;
+    lat[j] = a;
   }
   __syncthreads();
-  // W_uv: rank is a multiple of 32, 16-byte loads of eight weights; eight rows' loads are issued before the first is used
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int e0 = warp * 8; e0 < V; e0 += (MERGE_THREADS / 32) * 8) {
-    float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    for (int r = lane * 8; r < rank; r += 32 * 8) {
-      uint4 v[8];
+  // W_uv: rank is a multiple of 8, 16-byte loads of eight weights; the loads of ROWS rows are issued before the first is used
+  constexpr int ROWS = TT > 2 ? 4 : 8;
+  for (int e0 = warp * ROWS; e0 < V; e0 += (MERGE_THREADS / 32) * ROWS) {
+    float a[ROWS][TT];
 #pragma unroll
-      for (int k = 0; k < 8; ++k)
+    for (int k = 0; k < ROWS; ++k)
+#pragma unroll
+      for (int t = 0; t < TT; ++t) a[k][t] = 0.f;
+    for (int r = lane * 8; r < rank; r += 32 * 8) {
+      uint4 v[ROWS];
+#pragma unroll
+      for (int k = 0; k < ROWS; ++k)
         v[k] = e0 + k < V ? *reinterpret_cast<const uint4*>(w_uv + ((size_t)h * V + e0 + k) * rank + r) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&v[k]);
+      for (int t = 0; t < TT; ++t) {
+        float x[8];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          const float2 f = __bfloat1622float2(p[c]);
-          a[k] = fmaf(f.x, lat[r + 2 * c], a[k]);
-          a[k] = fmaf(f.y, lat[r + 2 * c + 1], a[k]);
+        for (int c = 0; c < 8; ++c) x[c] = lat[t * rank + r + c];
+#pragma unroll
+        for (int k = 0; k < ROWS; ++k) {
+          const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&v[k]);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const float2 f = __bfloat1622float2(p[c]);
+            a[k][t] = fmaf(f.x, x[2 * c], a[k][t]);
+            a[k][t] = fmaf(f.y, x[2 * c + 1], a[k][t]);
+          }
         }
       }
     }
 #pragma unroll
-    for (int k = 0; k < 8; ++k) {
-      const float sum = warp_sum(a[k]);
-      if (lane == 0 && e0 + k < V) o[e0 + k] = from_f32<T>(gate ? sum * gate[(size_t)t * H + h] : sum);
-    }
+    for (int k = 0; k < ROWS; ++k)
+#pragma unroll
+      for (int t = 0; t < TT; ++t) {
+        const float sum = warp_sum(a[k][t]);
+        if (lane == 0 && e0 + k < V && t < n_t)
+          out[((size_t)(t0 + t) * H + h) * V + e0 + k] = from_f32<T>(gate ? sum * gate[(size_t)(t0 + t) * H + h] : sum);
+      }
   }
 }
 
@@ -375,13 +408,36 @@ size_t decode_smem(int mt, int width) {
   return (size_t)(mt * 16 + BK) * (width + 8) * 2 + (size_t)mt * 16 * PLD * 2 + (size_t)8 * mt * 16 * 4;
 }
 
+bool umma_enabled() {
+  static const bool on = [] { const char* e = getenv("IERT_LATENT_UMMA"); return !(e && e[0] == '0'); }();
+  return on;
+}
+
 }  // namespace
 
+// latent_decode_umma.cu
+int latent_umma_heads(int H, int rank, int R);
+int launch_latent_decode_umma(const void* qa, const IertBatchView* batch, const IertKvView* kv, int H, int Hpad, int R, float scale,
+                              int splits, float* part_m, float* part_l, float* part_acc, int* err, cudaStream_t stream);
+
 // Heads padded to whole MMA tiles (16, or 32 from 17 heads on), and how many runs of tiles a sequence is cut into.
-IERT_API int iert_latent_decode_tc_plan(int n_seqs, int H, int table_width, int* Hpad, int* splits) {
+// `table_width`: pages of the longest walk.
+IERT_API int iert_latent_decode_tc_plan(int n_seqs, int H, int rank, int R, int table_width, int* Hpad, int* splits) {
   const int tiles = (H + 15) / 16, mt = tiles >= 2 ? 2 : 1;
   const int groups = (tiles + mt - 1) / mt;
   *Hpad = groups * mt * 16;
+  if (umma_enabled() && latent_umma_heads(H, rank, R)) {
+    // one CTA per SM: as many runs as end soonest, a run costing its pages and about two pages' worth of beginning and end
+    const int slots = iert_sm_count_cached(), ctas = n_seqs * groups > 0 ? n_seqs * groups : 1;
+    int best = 1;
+    long long best_cost = -1;
+    for (int k = 1; k <= 32; ++k) {
+      const long long cost = (long long)((ctas * k + slots - 1) / slots) * ((table_width + k - 1) / k + 2);
+      if (best_cost < 0 || cost < best_cost) { best = k; best_cost = cost; }
+    }
+    *splits = best;
+    return IERT_OK;
+  }
   int want = (2 * iert_sm_count_cached() + n_seqs * groups - 1) / (n_seqs * groups > 0 ? n_seqs * groups : 1);
   if (want > 32) want = 32;
   // a run's partial result (heads x rank floats) is as many bytes as 16 or more cached rows: runs of fewer than
@@ -404,9 +460,11 @@ IERT_API int iert_latent_attention_decode_tc(const void* q, int q_f32, long long
                                              cudaStream_t stream) {
   const int T = batch->n_tokens, width = kv->head_dim, rank = width - R;
   if (T <= 0) return IERT_OK;
-  if (T != batch->n_seqs || kv->dtype != IERT_BF16 || kv->kv_heads != 1 || kv->page_tokens != BK || rank % 32 || R < 0 ||
-      R % 16 || width > 640 || rank < 32 || rank > MAX_NTW * 32 || H <= 0 || Hpad % 16 || Hpad < H || Hpad > 65535 || splits < 1 || splits > 64 ||
-      D <= 0 || D > 8192 || V <= 0 || (q_f32 && R > 0 && !inv_freq))
+  const bool umma = umma_enabled() && latent_umma_heads(H, rank, R) && ((uintptr_t)qa & 15) == 0 && ((uintptr_t)kv->k & 15) == 0;
+  if (!umma && (rank % 32 || R % 16 || rank < 32)) return IERT_BAD_ARGUMENT;
+  if (T != batch->n_seqs || kv->dtype != IERT_BF16 || kv->kv_heads != 1 || kv->page_tokens != BK || rank % 8 || R < 0 ||
+      width > 640 || rank < 8 || rank > MAX_NTW * 32 || H <= 0 || Hpad % 16 || Hpad < H || Hpad > 65535 || splits < 1 || splits > 64 ||
+      D <= 0 || 4 * (D + 4 * rank) > 12000 || V <= 0 || (q_f32 && R > 0 && !inv_freq))
     return IERT_BAD_ARGUMENT;
   const int mt = Hpad % 32 == 0 ? 2 : 1;
   const size_t smem = decode_smem(mt, width);
@@ -420,23 +478,31 @@ IERT_API int iert_latent_attention_decode_tc(const void* q, int q_f32, long long
     }
     configured = true;
   }
-  const size_t absorb_smem = (size_t)(D + 4 * rank) * sizeof(float);
-  if (q_f32)
-    launch_dep(latent_absorb_q_kernel<float>, dim3(T, Hpad), dim3(ABSORB_THREADS), absorb_smem, stream, (const float*)q, ldq,
-               (const __nv_bfloat16*)w_uk, (__nv_bfloat16*)qa, H, Hpad, D, R, rank, inv_freq, rot_mul, pairing, *batch);
-  else
-    launch_dep(latent_absorb_q_kernel<__nv_bfloat16>, dim3(T, Hpad), dim3(ABSORB_THREADS), absorb_smem, stream,
-               (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)w_uk, (__nv_bfloat16*)qa, H, Hpad, D, R, rank, inv_freq, rot_mul,
-               pairing, *batch);
+  // tokens that share a head's weights in the kernels around: one when there are few, so that there are blocks enough
+  const int tt = T <= 4 ? 1 : T <= 8 ? 2 : 4;
+#define ABSORB(TQ, TT)                                                                                                             \
+  launch_dep(latent_absorb_q_kernel<TQ, TT>, dim3((T + TT - 1) / TT, Hpad), dim3(ABSORB_THREADS), (size_t)TT * (D + 4 * rank) * sizeof(float), \
+             stream, (const TQ*)q, ldq, (const __nv_bfloat16*)w_uk, (__nv_bfloat16*)qa, H, Hpad, D, R, rank, inv_freq, rot_mul, pairing, *batch)
+  if (q_f32) { if (tt == 1) ABSORB(float, 1); else if (tt == 2) ABSORB(float, 2); else ABSORB(float, 4); }
+  else { if (tt == 1) ABSORB(__nv_bfloat16, 1); else if (tt == 2) ABSORB(__nv_bfloat16, 2); else ABSORB(__nv_bfloat16, 4); }
+#undef ABSORB
   dim3 grid(T, splits, Hpad / (mt * 16));
-  if (mt == 2)
+  if (umma) {
+    const int st = launch_latent_decode_umma(qa, batch, kv, H, Hpad, R, scale, splits, part_m, part_l, part_acc, err, stream);
+    if (st != IERT_OK) return IERT_CUDA_ERROR;       // (the sizes were checked above)
+  } else if (mt == 2)
     launch_dep(latent_decode_tc_kernel<2>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16*)qa, *batch, *kv, Hpad, R,
                scale, splits, part_m, part_l, part_acc, err);
   else
     launch_dep(latent_decode_tc_kernel<1>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16*)qa, *batch, *kv, Hpad, R,
                scale, splits, part_m, part_l, part_acc, err);
-  launch_dep(latent_decode_merge_kernel<__nv_bfloat16>, dim3(T, H), dim3(MERGE_THREADS), (size_t)(rank + 64) * sizeof(float),
-             stream, (const float*)part_m, (const float*)part_l, (const float*)part_acc, splits, Hpad, rank, sink, gate,
-             (const __nv_bfloat16*)w_uv, (__nv_bfloat16*)out, *batch, H, V);
+#define MERGE(TT)                                                                                                                  \
+  launch_dep(latent_decode_merge_kernel<__nv_bfloat16, TT>, dim3((T + TT - 1) / TT, H), dim3(MERGE_THREADS),                       \
+             (size_t)TT * (rank + 64) * sizeof(float), stream, (const float*)part_m, (const float*)part_l, (const float*)part_acc, splits, \
+             Hpad, rank, sink, gate, (const __nv_bfloat16*)w_uv, (__nv_bfloat16*)out, *batch, H, V)
+  if (tt == 1) MERGE(1);
+  else if (tt == 2) MERGE(2);
+  else MERGE(4);
+#undef MERGE
   return iert_check_launch("latent_attention_decode_tc");
 }

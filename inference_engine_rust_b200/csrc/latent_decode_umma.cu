@@ -1,0 +1,407 @@
+// One-token steps of latent attention on the 5th-generation tensor cores: the attention over the cached rows, in the
+// absorbed form (latent_decode_tc.cu has the absorption of the queries before it and the merge behind it).  A cached row
+// [latent | rotated key part] is the key of every head and, in its latent part, the value of every head, so a page of 64
+// rows comes into shared memory once and is an operand of both products, with the HEADS as the narrow side of each:
+//
+//   S^T = C Qa^T    [keys x heads]   A = the page, K-major (its rows are the keys),       B = the absorbed queries
+//   L^T += C^T P^T  [rank x heads]   A = the same page, MN-major (its columns are rows),  B = the probabilities
+//
+//   A page has 64 rows and an instruction takes 128: the upper half of S^T is made from whatever lies behind the page in
+//   shared memory and is never read (a row of A only reaches its own row of D).
+//   grid (sequences, runs of pages, groups of NH heads); a CTA walks its run of the sequence's pages.
+//   warp 4      TMA producer: the queries once, then pages into a ring of `stages`; pages other than the newest one are
+//               asked for before the wait on the kernel in front.
+//   warp 5      MMA issuer: the scores of the next page as soon as it has landed, the weighted sum of this one as soon as
+//               its probabilities are there, whichever comes first.
+//   warps 0, 1  softmax, a key per thread (a row of S^T is a TMEM lane): mask, maximum per head over the page's keys by
+//               halving exchanges, exponentials against a reference maximum that moves only when it has grown by more
+//               than 2^8, probabilities as bf16 into (swizzled) shared memory.  A row that does not count (outside the
+//               window, beyond the newest position, a page that is not there) is cleared first: its weight is zero, but
+//               zero times whatever the page held need not be.
+//   warps 0-3   rescale L^T in TMEM when a reference maximum moves, and write the run's partial result at the end.
+//   Every wait is bounded; on expiry the kernel records IERT_ERR_WAIT_EXPIRED, waits (bounded) for its copies and MMAs,
+//   frees its TMEM and returns.
+#include "common.cuh"
+#include "sm100.cuh"
+#include "tma_host.cuh"
+
+using namespace iert;
+using namespace sm100;
+
+namespace {
+
+constexpr int BK = 64;                         // keys per page
+constexpr int BOX = BK * 128;                  // 64 rows x 64 columns of bf16
+constexpr int THREADS = 192, SOFT = 128;
+constexpr uint32_t WAIT_LIMIT = 1u << 22;
+constexpr int MAX_STAGES = 4;
+
+struct LatentUmmaParams {
+  int Hpad, H, rank, nbox, ksteps, mblocks, splits, stages;
+  uint32_t tmem_cols;
+  float scale_log2e;
+  float* part_m;
+  float* part_l;
+  float* part_acc;
+  int* err;
+};
+
+__device__ __forceinline__ bool wait_bar(uint64_t* bar, uint32_t parity, volatile int* abort_flag) {
+  for (uint32_t i = 0; i < WAIT_LIMIT; ++i) {
+    if (mbar_try_wait(bar, parity)) return true;
+    if ((i & 255u) == 255u && *abort_flag) return false;
+  }
+  return false;
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void soft_sync() { asm volatile("bar.sync 1, %0;" ::"n"(SOFT) : "memory"); }
+
+// v[0 .. N) of every lane combined over the warp: lane l gets element l % N.  Each exchange halves what a lane still holds.
+template <int N, bool MAX>
+__device__ __forceinline__ float reduce_columns(float (&v)[N], int lane) {
+#pragma unroll
+  for (int n = N / 2; n > 0; n /= 2) {
+    const bool upper = (lane & n) != 0;
+#pragma unroll
+    for (int i = 0; i < n; ++i) {
+      const float keep = upper ? v[i + n] : v[i], send = upper ? v[i] : v[i + n];
+      const float got = __shfl_xor_sync(0xffffffffu, send, n);
+      v[i] = MAX ? fmaxf(keep, got) : keep + got;
+    }
+  }
+  if (N < 32) {
+    const float got = __shfl_xor_sync(0xffffffffu, v[0], 16);
+    v[0] = MAX ? fmaxf(v[0], got) : v[0] + got;
+  }
+  return v[0];
+}
+
+template <int NH>
+__global__ void __launch_bounds__(THREADS, 1)
+latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_constant__ CUtensorMap map_q, LatentUmmaParams p,
+                          IertBatchView b, IertKvView kv) {
+  extern __shared__ __align__(1024) uint8_t smem[];     // no static shared memory: the window starts 1024-byte aligned
+  constexpr int QBOX = NH * 128, PBUF = NH * 128;
+  uint8_t* q_s = smem;                                   // nbox boxes of NH rows
+  uint8_t* c_s = q_s + p.nbox * QBOX;                    // stages x nbox boxes of 64 rows
+  uint8_t* p_s = c_s + p.stages * p.nbox * BOX;          // 2 buffers: NH rows (heads) of 64 probabilities
+  uint8_t* tail = p_s + (2 * PBUF > BOX ? 2 * PBUF : BOX);      // (an MMA may read one box beyond the last page)
+  float* wmax = reinterpret_cast<float*>(tail);          // [2][2][NH]
+  float* wsum = wmax + 4 * NH;                           // [NH]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(wsum + NH);
+  uint64_t* q_full = bars;
+  uint64_t* c_full = bars + 1;                           // MAX_STAGES
+  uint64_t* c_empty = c_full + MAX_STAGES;               // MAX_STAGES
+  uint64_t* s_full = c_empty + MAX_STAGES;               // 2
+  uint64_t* p_ready = s_full + 2;                        // 2
+  uint64_t* pv_done = p_ready + 2;                       // 2
+  uint64_t* drained = pv_done + 2;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(drained + 1);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  volatile int* armed = abort_flag + 1;                  // pages the producer has asked for; -1: not even the queries
+  volatile int* stop = armed + 1;                        // [2]: the flag as warp 0 saw it in front of a barrier, so that all agree
+
+  const int s = blockIdx.x, split = blockIdx.y, rows0 = blockIdx.z * NH;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_launch_dependents();
+  const int slot = b.slot_ids[s];
+  if (slot < 0) { pdl_wait(); return; }
+  const int pos = b.pos0[s];                             // one token per sequence: its own row is in the cache
+  const IertPageWalk walk = iert_page_walk(kv, pos, BK);
+  const int t_lo = (int)((long long)split * walk.n / p.splits), t_hi = (int)((long long)(split + 1) * walk.n / p.splits);
+  const int n_tiles = t_hi - t_lo;
+  const size_t part_row0 = ((size_t)s * p.splits + split) * p.Hpad + rows0;
+  if (n_tiles <= 0) {                                    // an empty run: a partial that the merge skips
+    pdl_wait();
+    if (tid < NH) { p.part_m[part_row0 + tid] = -INFINITY; p.part_l[part_row0 + tid] = 0.f; }
+    return;
+  }
+  if (smem_addr(smem) & 1023u) {                         // never expected; refuse rather than compute garbage
+    if (tid == 0) atomicOr(p.err, IERT_ERR_WAIT_EXPIRED);
+    return;
+  }
+  if (tid == 0) {
+    mbar_init(q_full, 1);
+    for (int i = 0; i < MAX_STAGES; ++i) { mbar_init(&c_full[i], 1); mbar_init(&c_empty[i], 1); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_ready[i], SOFT); mbar_init(&pv_done[i], 1); }
+    mbar_init(drained, 1);
+    *abort_flag = 0;
+    *armed = -1;
+    mbar_fence_init();
+    tma_prefetch_desc(&map_c);
+    tma_prefetch_desc(&map_q);
+  }
+  if (warp == 5) tmem_alloc(tmem_slot, p.tmem_cols);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  const uint32_t l_col = 2 * NH;                         // S^T buffers at columns 0 and NH, the blocks of L^T behind them
+  bool ok = true;
+
+  if (warp == 4) {
+    // ---------------- TMA producer ----------------
+    bool waited = false;
+    int asked = 0;
+    for (int base = 0; base < n_tiles; base += 32) {
+      int page = -1;                                     // page numbers of up to 32 pages at a time, one per lane
+      if (base + lane < n_tiles)
+        page = kv.page_table[(size_t)slot * kv.table_width + iert_table_entry(kv, iert_walk_page(walk, t_lo + base + lane))];
+      for (int k = 0; k < 32 && base + k < n_tiles; ++k) {
+        const int it = base + k, st = it % p.stages;
+        const int pgid = __shfl_sync(0xffffffffu, page, k);
+        if (lane != 0 || !ok) continue;
+        // the newest row, and the queries, are the work of the kernels in front
+        if (!waited && (t_lo + it == walk.n - 1 || it >= p.stages)) {
+          pdl_wait();
+          waited = true;
+          mbar_expect_tx(q_full, p.nbox * QBOX);
+          for (int x = 0; x < p.nbox; ++x) tma_load_2d(q_s + x * QBOX, &map_q, q_full, 64 * x, s * p.Hpad + rows0);
+        }
+        if (it >= p.stages && !wait_bar(&c_empty[st], ((it / p.stages) - 1) & 1, abort_flag)) { ok = false; continue; }
+        const bool page_ok = pgid >= 0 && pgid < kv.n_pages;
+        if (!page_ok) atomicOr(p.err, IERT_ERR_PAGE_RANGE);      // (the softmax warps see the same and count no row of it)
+        mbar_expect_tx(&c_full[st], p.nbox * BOX);
+        for (int x = 0; x < p.nbox; ++x)
+          tma_load_2d(c_s + (st * p.nbox + x) * BOX, &map_c, &c_full[st], 64 * x, (page_ok ? pgid : 0) * BK);
+        asked = it + 1;
+      }
+    }
+    if (lane == 0) {
+      if (!waited) {
+        pdl_wait();
+        waited = true;
+        mbar_expect_tx(q_full, p.nbox * QBOX);
+        for (int x = 0; x < p.nbox; ++x) tma_load_2d(q_s + x * QBOX, &map_q, q_full, 64 * x, s * p.Hpad + rows0);
+      }
+      *armed = asked;
+    }
+  } else if (warp == 5) {
+    // ---------------- MMA issuer ----------------
+    if (lane == 0) {
+      constexpr uint32_t IDESC_S = instr_desc_bf16(128, NH);
+      constexpr uint32_t IDESC_L = instr_desc_bf16_a_mn(128, NH);
+      auto scores = [&](int it) {                        // S^T[it & 1] = C_it Qa^T (the page has landed)
+        const int st = it % p.stages;
+        tc_fence_after();
+        const uint32_t cb = smem_addr(c_s + st * p.nbox * BOX), qb = smem_addr(q_s);
+        for (int ks = 0; ks < p.ksteps; ++ks)
+          umma_bf16(tmem + (it & 1) * NH, smem_desc_k128(cb + (ks / 4) * BOX + (ks % 4) * 32),
+                    smem_desc_k128(qb + (ks / 4) * QBOX + (ks % 4) * 32), IDESC_S, ks > 0 ? 1u : 0u);
+        umma_commit(&s_full[it & 1]);
+      };
+      ok = wait_bar(q_full, 0, abort_flag) && wait_bar(&c_full[0], 0, abort_flag);
+      if (ok) scores(0);
+      for (int it = 0; ok && it < n_tiles; ++it) {
+        const int st = it % p.stages, nx = it + 1, sn = nx % p.stages;
+        bool next_done = nx >= n_tiles, ready = false;
+        for (uint32_t i = 0; i < WAIT_LIMIT && !ready; ++i) {
+          if (!next_done && mbar_try_wait(&c_full[sn], (nx / p.stages) & 1)) { scores(nx); next_done = true; }
+          ready = mbar_try_wait(&p_ready[it & 1], (it >> 1) & 1);
+          if ((i & 255u) == 255u && *abort_flag) break;
+        }
+        if (!ready) { ok = false; break; }
+        tc_fence_after();
+        const uint32_t cb = smem_addr(c_s + st * p.nbox * BOX), pb = smem_addr(p_s + (it & 1) * PBUF);
+        for (int m = 0; m < p.mblocks; ++m)
+#pragma unroll
+          for (int kk = 0; kk < BK / 16; ++kk)
+            umma_bf16(tmem + l_col + m * NH, smem_desc_mn128(cb + 2 * m * BOX + kk * 16 * 128, BOX), smem_desc_k128(pb + kk * 32),
+                      IDESC_L, (it > 0 || kk > 0) ? 1u : 0u);
+        umma_commit(&pv_done[it & 1]);
+        umma_commit(&c_empty[st]);
+        if (!next_done) {
+          if (!wait_bar(&c_full[sn], (nx / p.stages) & 1, abort_flag)) { ok = false; break; }
+          scores(nx);
+        }
+      }
+      umma_commit(drained);
+    }
+  } else {
+    // ---------------- softmax, rescaling ----------------
+    pdl_wait();
+    const uint32_t lane_bits = (uint32_t)(warp * 32) << 16;
+    const int row = tid;                                 // the key of the page, for warps 0 and 1
+    float m_ref = -INFINITY;                             // lane h: the reference maximum of head h % NH (base 2), alike in all warps
+    float l[NH];
+#pragma unroll
+    for (int h = 0; h < NH; ++h) l[h] = 0.f;
+    for (int it = 0; it < n_tiles; ++it) {
+      float sc[NH];
+      if (warp < 2) {
+        const int pg = iert_walk_page(walk, t_lo + it), j = pg * BK + row;
+        const int page = kv.page_table[(size_t)slot * kv.table_width + iert_table_entry(kv, pg)];
+        const bool vis = page >= 0 && page < kv.n_pages && j <= pos && (j >= walk.j_min || j < kv.keep);
+        if (!wait_bar(&s_full[it & 1], (it >> 1) & 1, abort_flag)) ok = false;
+        tc_fence_after();
+        uint32_t raw[NH];
+#pragma unroll
+        for (int c = 0; c < NH; c += 16) tmem_ld16_issue(tmem + lane_bits + (it & 1) * NH + c, raw + c);
+        tmem_ld_wait();
+        float mx[NH];
+#pragma unroll
+        for (int h = 0; h < NH; ++h) mx[h] = sc[h] = vis ? __uint_as_float(raw[h]) * p.scale_log2e : -INFINITY;
+        if (!vis) {
+          uint8_t* line = c_s + (it % p.stages) * p.nbox * BOX + row * 128;
+          for (int x = 0; x < p.nbox; ++x)
+#pragma unroll
+            for (int c = 0; c < 8; ++c) *reinterpret_cast<uint4*>(line + x * BOX + c * 16) = make_uint4(0u, 0u, 0u, 0u);
+        }
+        __syncwarp();
+        const float top = reduce_columns<NH, true>(mx, lane);
+        if (lane < NH) wmax[((it & 1) * 2 + warp) * NH + lane] = top;
+        if (!ok) *abort_flag = 1;
+      }
+      if (tid == 0) stop[it & 1] = *abort_flag;
+      soft_sync();
+      if (stop[it & 1]) { ok = false; break; }           // all four warps leave at the same barrier
+      const int hl = lane % NH;
+      const float tm = fmaxf(wmax[(it & 1) * 2 * NH + hl], wmax[((it & 1) * 2 + 1) * NH + hl]);
+      const bool grow = tm > m_ref + 8.0f || (m_ref == -INFINITY && tm != -INFINITY);
+      if (__any_sync(0xffffffffu, grow)) {               // the same in all four warps
+        const float m_new = grow ? tm : m_ref;
+        const float alpha = !grow ? 1.f : (m_ref == -INFINITY ? 0.f : ex2(m_ref - m_new));
+        m_ref = m_new;
+#pragma unroll
+        for (int h = 0; h < NH; ++h) l[h] *= __shfl_sync(0xffffffffu, alpha, h);
+        if (it > 0) {
+          if (!wait_bar(&pv_done[(it - 1) & 1], ((it - 1) >> 1) & 1, abort_flag)) { ok = false; *abort_flag = 1; }
+          tc_fence_after();
+          for (int m = 0; m < p.mblocks; ++m)
+#pragma unroll
+            for (int c = 0; c < NH; c += 16) {
+              float o[16];
+              tmem_ld16(tmem + lane_bits + l_col + m * NH + c, o);
+#pragma unroll
+              for (int e = 0; e < 16; ++e) o[e] *= __shfl_sync(0xffffffffu, alpha, c + e);
+              tmem_st16(tmem + lane_bits + l_col + m * NH + c, o);
+            }
+        }
+      }
+      if (warp < 2) {
+        // probabilities: head h is row h of the operand, key `row` its column; the buffer was last read by the sum of page
+        // it - 2, which had finished before the scores of page `it` were committed
+        uint8_t* pb = p_s + (it & 1) * PBUF + (row & 7) * 2;
+        const float neg = m_ref == -INFINITY ? 0.f : -m_ref;
+#pragma unroll
+        for (int h = 0; h < NH; ++h) {
+          const float pr = ex2(sc[h] + __shfl_sync(0xffffffffu, neg, h));
+          l[h] += pr;
+          *reinterpret_cast<__nv_bfloat16*>(pb + h * 128 + (((row >> 3) ^ (h & 7)) << 4)) = __float2bfloat16_rn(pr);
+        }
+        fence_proxy_async_smem();                        // the probabilities, and rows that were cleared, reach the tensor core
+      }
+      tc_fence_before();
+      mbar_arrive(&p_ready[it & 1]);
+    }
+    if (ok && !wait_bar(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, abort_flag)) ok = false;
+    __syncwarp();
+    const float lw = reduce_columns<NH, false>(l, lane);     // (warps 2 and 3 hold zeros)
+    if (ok && warp == 1 && lane < NH) wsum[lane] = lw;
+    if (!ok) *abort_flag = 1;
+    soft_sync();                                         // every warp has left the loop and said how
+    if (tid == 0) stop[0] = *abort_flag;
+    soft_sync();
+    const bool good = stop[0] == 0;                      // an aborted run leaves an empty partial
+    if (warp == 0 && lane < NH) {
+      p.part_m[part_row0 + lane] = good && m_ref != -INFINITY ? m_ref * 0.6931471805599453f : -INFINITY;
+      p.part_l[part_row0 + lane] = good ? lw + wsum[lane] : 0.f;
+    }
+    if (good) {
+      tc_fence_after();
+      for (int m = 0; m < p.mblocks; ++m) {
+        const int r = m * 128 + tid;
+#pragma unroll
+        for (int c = 0; c < NH; c += 16) {
+          float o[16];
+          tmem_ld16(tmem + lane_bits + l_col + m * NH + c, o);
+#pragma unroll
+          for (int e = 0; e < 16; ++e)
+            if (r < p.rank && rows0 + c + e < p.H) p.part_acc[(part_row0 + c + e) * p.rank + r] = o[e];
+        }
+      }
+    }
+  }
+  if (!ok && lane == 0) {
+    atomicOr(p.err, IERT_ERR_WAIT_EXPIRED);
+    *abort_flag = 1;
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_flag && tid == 0) {                         // copies and MMAs still on their way end before the memory is let go
+    mbar_wait(drained, 0, WAIT_LIMIT);
+    const int n = *armed;
+    if (n >= 0) mbar_wait(q_full, 0, WAIT_LIMIT);
+    for (int st = 0; st < p.stages; ++st)
+      if (n > st) {
+        const int last = ((n - 1 - st) / p.stages) * p.stages + st;
+        mbar_wait(&c_full[st], (last / p.stages) & 1, WAIT_LIMIT);
+      }
+  }
+  __syncthreads();
+  if (warp == 5) {
+    tc_fence_after();
+    tmem_dealloc(tmem, p.tmem_cols);
+  }
+}
+
+size_t fixed_smem(int nh, int nbox) {
+  const size_t pbuf = (size_t)nh * 128;
+  return (size_t)nbox * nh * 128 + (2 * pbuf > (size_t)BOX ? 2 * pbuf : (size_t)BOX) + (4 * nh + nh) * sizeof(float) +
+         (2 + 2 * MAX_STAGES + 6) * sizeof(uint64_t) + 64;
+}
+int stages_for(int nh, int width) {
+  const int nbox = (width + 63) / 64;
+  const size_t room = 227 * 1024 - fixed_smem(nh, nbox);
+  const int n = (int)(room / ((size_t)nbox * BOX));
+  return n > MAX_STAGES ? MAX_STAGES : n;
+}
+
+}  // namespace
+
+// Heads per CTA (16 or 32) that the kernel runs at H heads, or 0 where it does not take the sizes.
+int latent_umma_heads(int H, int rank, int R) {
+  const int width = rank + R, nh = H > 16 ? 32 : 16;
+  if (width % 8 || rank < 16 || rank > 512 || width > 640 || stages_for(nh, width) < 2) return 0;
+  return nh;
+}
+
+// qa bf16 [T, Hpad, width]; part_m, part_l fp32 [T, splits, Hpad]; part_acc fp32 [T, splits, Hpad, rank] (rows of heads below
+// H are written).  One token per sequence; a cache of bf16 rows `width` = rank + R wide, pages of 64.
+int launch_latent_decode_umma(const void* qa, const IertBatchView* batch, const IertKvView* kv, int H, int Hpad, int R, float scale,
+                              int splits, float* part_m, float* part_l, float* part_acc, int* err, cudaStream_t stream) {
+  const int T = batch->n_tokens, width = kv->head_dim, rank = width - R;
+  const int nh = latent_umma_heads(H, rank, R);
+  if (!nh || Hpad % nh || ((uintptr_t)qa & 15) || ((uintptr_t)kv->k & 15)) return IERT_BAD_ARGUMENT;
+  CUtensorMap map_c, map_q;
+  if (!tma_host::tensor_map_2d(kv->k, (long long)kv->n_pages * BK, width, width, BK, &map_c) ||
+      !tma_host::tensor_map_2d(qa, (long long)T * Hpad, width, width, nh, &map_q))
+    return IERT_BAD_ARGUMENT;
+  LatentUmmaParams p;
+  p.Hpad = Hpad; p.H = H; p.rank = rank;
+  p.nbox = (width + 63) / 64; p.ksteps = (width + 15) / 16; p.mblocks = (rank + 127) / 128;
+  p.splits = splits; p.stages = stages_for(nh, width);
+  const int cols = 2 * nh + p.mblocks * nh;
+  p.tmem_cols = 32;
+  while ((int)p.tmem_cols < cols) p.tmem_cols *= 2;
+  p.scale_log2e = scale * 1.4426950408889634f;
+  p.part_m = part_m; p.part_l = part_l; p.part_acc = part_acc; p.err = err;
+  const size_t smem = fixed_smem(nh, p.nbox) + (size_t)p.stages * p.nbox * BOX;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(latent_decode_umma_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(latent_decode_umma_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) {
+      cudaGetLastError();
+      return IERT_CUDA_ERROR;
+    }
+    configured = true;
+  }
+  const dim3 grid(T, splits, Hpad / nh);
+  if (nh == 16) launch_dep(latent_decode_umma_kernel<16>, grid, dim3(THREADS), smem, stream, map_c, map_q, p, *batch, *kv);
+  else launch_dep(latent_decode_umma_kernel<32>, grid, dim3(THREADS), smem, stream, map_c, map_q, p, *batch, *kv);
+  return cudaGetLastError() == cudaSuccess ? IERT_OK : IERT_CUDA_ERROR;
+}

@@ -229,4 +229,9 @@ __host__ __device__ constexpr uint32_t instr_desc_bf16_b_mn(uint32_t M, uint32_t
   return instr_desc_bf16(M, N) | (1u << 16);
 }
 
+// The same with the A operand MN-major (bit 15).
+__host__ __device__ constexpr uint32_t instr_desc_bf16_a_mn(uint32_t M, uint32_t N) {
+  return instr_desc_bf16(M, N) | (1u << 15);
+}
+
 }  // namespace sm100

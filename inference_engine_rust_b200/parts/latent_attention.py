@@ -194,7 +194,7 @@ class LatentAttention(Mixer):
             done = False
             if rt.fast and c_ext.dtype == torch.bfloat16 and ctx.kind == "decode":
                 group = cache_view.group
-                hpad, splits = B.latent_decode_tc_plan(ctx.n_seqs, H, min(group.table_width, group.ring_pages + 1))
+                hpad, splits = B.latent_decode_tc_plan(ctx.n_seqs, H, rank, R, min(group.table_width, group.ring_pages + 1))
                 qa = ws.take("latent.qa", (T, hpad, rank + R), torch.bfloat16)
                 part_m = ws.take("latent.part_m", (T, splits, hpad), torch.float32)
                 part_l = ws.take("latent.part_l", (T, splits, hpad), torch.float32)
@@ -237,7 +237,7 @@ class LatentAttention(Mixer):
             self.uq.apply(cq, q, T, ctx.stream)
             done = False
             if rt.fast and q.dtype == torch.bfloat16 and ctx.kind == "decode":
-                hpad, splits = B.latent_decode_tc_plan(ctx.n_seqs, H, cache_view.group.table_width)
+                hpad, splits = B.latent_decode_tc_plan(ctx.n_seqs, H, self.kv_rank, 0, cache_view.group.table_width)
                 rank = self.kv_rank
                 qa = ws.take("latent.qa", (T, hpad, rank), torch.bfloat16)
                 part_m = ws.take("latent.part_m", (T, splits, hpad), torch.float32)
