@@ -1,24 +1,25 @@
 // One-token steps of latent attention on the 5th-generation tensor cores: the attention over the cached rows, in the
 // absorbed form (latent_decode_tc.cu has the absorption of the queries before it and the merge behind it).  A cached row
 // [latent | rotated key part] is the key of every head and, in its latent part, the value of every head, so a page of 64
-// rows comes into shared memory once and is an operand of both products, with the HEADS as the narrow side of each:
+// rows comes into shared memory once and is an operand of both products:
 //
-//   S^T = C Qa^T    [keys x heads]   A = the page, K-major (its rows are the keys),       B = the absorbed queries
+//   S = Qa C^T      [heads x keys]   A = the absorbed queries, from tensor memory,       B = the page, K-major
 //   L^T += C^T P^T  [rank x heads]   A = the same page, MN-major (its columns are rows),  B = the probabilities
 //
-//   A page has 64 rows and an instruction takes 128: the upper half of S^T is made from whatever lies behind the page in
-//   shared memory and is never read (a row of A only reaches its own row of D).
+//   What an instruction costs here is the shared memory it reads (about 64 bytes a cycle), so the queries, which every
+//   page meets, live in TMEM: 128 lanes hold 128 / NH copies of the NH heads, every warp of the softmax finds all heads in
+//   its own 32 lanes and takes 16 of the page's 64 keys.  Their way there is through the last stage of the page ring,
+//   which is filled with pages once they have moved on.
 //   grid (sequences, runs of pages, groups of NH heads); a CTA walks its run of the sequence's pages.
-//   warp 4      TMA producer: the queries once, then pages into a ring of `stages`; pages other than the newest one are
-//               asked for before the wait on the kernel in front.
+//   warp 4      TMA producer: the queries once, then pages into a ring of `stages`; the first pages, unless one is the
+//               newest, are asked for before the wait on the kernel in front.
 //   warp 5      MMA issuer: the scores of the next page as soon as it has landed, the weighted sum of this one as soon as
 //               its probabilities are there, whichever comes first.
-//   warps 0, 1  softmax, a key per thread (a row of S^T is a TMEM lane): mask, maximum per head over the page's keys by
-//               halving exchanges, exponentials against a reference maximum that moves only when it has grown by more
-//               than 2^8, probabilities as bf16 into (swizzled) shared memory.  A row that does not count (outside the
-//               window, beyond the newest position, a page that is not there) is cleared first: its weight is zero, but
-//               zero times whatever the page held need not be.
-//   warps 0-3   rescale L^T in TMEM when a reference maximum moves, and write the run's partial result at the end.
+//   warps 0-3   softmax, a head per lane and 16 keys per warp: mask, the page's maximum per head through shared memory,
+//               exponentials against a reference maximum that moves only when it has grown by more than 2^8 (L^T is
+//               rescaled in TMEM then), probabilities as bf16 into (swizzled) shared memory.  A row of the page that does
+//               not count (outside the window, beyond the newest position, a page that is not there) is cleared first: its
+//               weight is zero, but zero times whatever the page held need not be.
 //   Every wait is bounded; on expiry the kernel records IERT_ERR_WAIT_EXPIRED, waits (bounded) for its copies and MMAs,
 //   frees its TMEM and returns.
 #include "common.cuh"
@@ -37,7 +38,7 @@ constexpr uint32_t WAIT_LIMIT = 1u << 22;
 constexpr int MAX_STAGES = 4;
 
 struct LatentUmmaParams {
-  int Hpad, H, rank, nbox, ksteps, mblocks, splits, stages;
+  int Hpad, H, rank, nbox, ksteps, qcols, mblocks, splits, stages;
   uint32_t tmem_cols;
   float scale_log2e;
   float* part_m;
@@ -60,44 +61,26 @@ __device__ __forceinline__ float ex2(float x) {
 }
 __device__ __forceinline__ void soft_sync() { asm volatile("bar.sync 1, %0;" ::"n"(SOFT) : "memory"); }
 
-// v[0 .. N) of every lane combined over the warp: lane l gets element l % N.  Each exchange halves what a lane still holds.
-template <int N, bool MAX>
-__device__ __forceinline__ float reduce_columns(float (&v)[N], int lane) {
-#pragma unroll
-  for (int n = N / 2; n > 0; n /= 2) {
-    const bool upper = (lane & n) != 0;
-#pragma unroll
-    for (int i = 0; i < n; ++i) {
-      const float keep = upper ? v[i + n] : v[i], send = upper ? v[i] : v[i + n];
-      const float got = __shfl_xor_sync(0xffffffffu, send, n);
-      v[i] = MAX ? fmaxf(keep, got) : keep + got;
-    }
-  }
-  if (N < 32) {
-    const float got = __shfl_xor_sync(0xffffffffu, v[0], 16);
-    v[0] = MAX ? fmaxf(v[0], got) : v[0] + got;
-  }
-  return v[0];
-}
-
 template <int NH>
 __global__ void __launch_bounds__(THREADS, 1)
 latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __grid_constant__ CUtensorMap map_q, LatentUmmaParams p,
                           IertBatchView b, IertKvView kv) {
   extern __shared__ __align__(1024) uint8_t smem[];     // no static shared memory: the window starts 1024-byte aligned
   constexpr int QBOX = NH * 128, PBUF = NH * 128;
-  uint8_t* q_s = smem;                                   // nbox boxes of NH rows
-  uint8_t* c_s = q_s + p.nbox * QBOX;                    // stages x nbox boxes of 64 rows
+  uint8_t* c_s = smem;                                   // stages x nbox boxes of 64 rows
+  uint8_t* q_s = c_s + (p.stages - 1) * p.nbox * BOX;    // nbox boxes of NH rows, in the last stage until they are in TMEM
   uint8_t* p_s = c_s + p.stages * p.nbox * BOX;          // 2 buffers: NH rows (heads) of 64 probabilities
   uint8_t* tail = p_s + (2 * PBUF > BOX ? 2 * PBUF : BOX);      // (an MMA may read one box beyond the last page)
-  float* wmax = reinterpret_cast<float*>(tail);          // [2][2][NH]
-  float* wsum = wmax + 4 * NH;                           // [NH]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(wsum + NH);
+  float* wmax = reinterpret_cast<float*>(tail);          // [2][4][32]
+  float* wsum = wmax + 8 * 32;                           // [4][32]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(wsum + 4 * 32);
   uint64_t* q_full = bars;
   uint64_t* c_full = bars + 1;                           // MAX_STAGES
   uint64_t* c_empty = c_full + MAX_STAGES;               // MAX_STAGES
-  uint64_t* s_full = c_empty + MAX_STAGES;               // 2
-  uint64_t* p_ready = s_full + 2;                        // 2
+  uint64_t* q_moved = c_empty + MAX_STAGES;              // the queries are in TMEM
+  uint64_t* s_full = q_moved + 1;
+  uint64_t* s_empty = s_full + 1;                        // every thread has read its scores
+  uint64_t* p_ready = s_empty + 1;                       // 2
   uint64_t* pv_done = p_ready + 2;                       // 2
   uint64_t* drained = pv_done + 2;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(drained + 1);
@@ -107,7 +90,6 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
 
   const int s = blockIdx.x, split = blockIdx.y, rows0 = blockIdx.z * NH;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  pdl_launch_dependents();
   const int slot = b.slot_ids[s];
   if (slot < 0) { pdl_wait(); return; }
   const int pos = b.pos0[s];                             // one token per sequence: its own row is in the cache
@@ -127,7 +109,10 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
   if (tid == 0) {
     mbar_init(q_full, 1);
     for (int i = 0; i < MAX_STAGES; ++i) { mbar_init(&c_full[i], 1); mbar_init(&c_empty[i], 1); }
-    for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_ready[i], SOFT); mbar_init(&pv_done[i], 1); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&p_ready[i], SOFT); mbar_init(&pv_done[i], 1); }
+    mbar_init(q_moved, SOFT);
+    mbar_init(s_full, 1);
+    mbar_init(s_empty, SOFT);
     mbar_init(drained, 1);
     *abort_flag = 0;
     *armed = -1;
@@ -139,8 +124,9 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  pdl_launch_dependents();                               // (a later kernel must not take the TMEM this CTA still waits for)
   const uint32_t tmem = *tmem_slot;
-  const uint32_t l_col = 2 * NH;                         // S^T buffers at columns 0 and NH, the blocks of L^T behind them
+  const uint32_t s_col = p.qcols, l_col = s_col + BK;    // the queries, S, and the blocks of L^T
   bool ok = true;
 
   if (warp == 4) {
@@ -156,12 +142,13 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
         const int pgid = __shfl_sync(0xffffffffu, page, k);
         if (lane != 0 || !ok) continue;
         // the newest row, and the queries, are the work of the kernels in front
-        if (!waited && (t_lo + it == walk.n - 1 || it >= p.stages)) {
+        if (!waited && (t_lo + it == walk.n - 1 || it >= p.stages - 1)) {
           pdl_wait();
           waited = true;
           mbar_expect_tx(q_full, p.nbox * QBOX);
           for (int x = 0; x < p.nbox; ++x) tma_load_2d(q_s + x * QBOX, &map_q, q_full, 64 * x, s * p.Hpad + rows0);
         }
+        if (it == p.stages - 1 && !wait_bar(q_moved, 0, abort_flag)) { ok = false; continue; }
         if (it >= p.stages && !wait_bar(&c_empty[st], ((it / p.stages) - 1) & 1, abort_flag)) { ok = false; continue; }
         const bool page_ok = pgid >= 0 && pgid < kv.n_pages;
         if (!page_ok) atomicOr(p.err, IERT_ERR_PAGE_RANGE);      // (the softmax warps see the same and count no row of it)
@@ -183,24 +170,25 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
   } else if (warp == 5) {
     // ---------------- MMA issuer ----------------
     if (lane == 0) {
-      constexpr uint32_t IDESC_S = instr_desc_bf16(128, NH);
+      constexpr uint32_t IDESC_S = instr_desc_bf16(128, BK);
       constexpr uint32_t IDESC_L = instr_desc_bf16_a_mn(128, NH);
-      auto scores = [&](int it) {                        // S^T[it & 1] = C_it Qa^T (the page has landed)
-        const int st = it % p.stages;
+      auto scores = [&](int it) {                        // S = Qa C_it^T (the page has landed, the scores before are read)
         tc_fence_after();
-        const uint32_t cb = smem_addr(c_s + st * p.nbox * BOX), qb = smem_addr(q_s);
+        const uint32_t cb = smem_addr(c_s + (it % p.stages) * p.nbox * BOX);
         for (int ks = 0; ks < p.ksteps; ++ks)
-          umma_bf16(tmem + (it & 1) * NH, smem_desc_k128(cb + (ks / 4) * BOX + (ks % 4) * 32),
-                    smem_desc_k128(qb + (ks / 4) * QBOX + (ks % 4) * 32), IDESC_S, ks > 0 ? 1u : 0u);
-        umma_commit(&s_full[it & 1]);
+          umma_bf16_a_tmem(tmem + s_col, tmem + ks * 8, smem_desc_k128(cb + (ks / 4) * BOX + (ks % 4) * 32), IDESC_S, ks > 0 ? 1u : 0u);
+        umma_commit(s_full);
       };
-      ok = wait_bar(q_full, 0, abort_flag) && wait_bar(&c_full[0], 0, abort_flag);
+      ok = wait_bar(q_moved, 0, abort_flag) && wait_bar(&c_full[0], 0, abort_flag);
       if (ok) scores(0);
       for (int it = 0; ok && it < n_tiles; ++it) {
         const int st = it % p.stages, nx = it + 1, sn = nx % p.stages;
         bool next_done = nx >= n_tiles, ready = false;
         for (uint32_t i = 0; i < WAIT_LIMIT && !ready; ++i) {
-          if (!next_done && mbar_try_wait(&c_full[sn], (nx / p.stages) & 1)) { scores(nx); next_done = true; }
+          if (!next_done && mbar_try_wait(s_empty, it & 1) && mbar_try_wait(&c_full[sn], (nx / p.stages) & 1)) {
+            scores(nx);
+            next_done = true;
+          }
           ready = mbar_try_wait(&p_ready[it & 1], (it >> 1) & 1);
           if ((i & 255u) == 255u && *abort_flag) break;
         }
@@ -215,61 +203,75 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
         umma_commit(&pv_done[it & 1]);
         umma_commit(&c_empty[st]);
         if (!next_done) {
-          if (!wait_bar(&c_full[sn], (nx / p.stages) & 1, abort_flag)) { ok = false; break; }
+          if (!wait_bar(s_empty, it & 1, abort_flag) || !wait_bar(&c_full[sn], (nx / p.stages) & 1, abort_flag)) { ok = false; break; }
           scores(nx);
         }
       }
       umma_commit(drained);
     }
   } else {
-    // ---------------- softmax, rescaling ----------------
+    // ---------------- softmax: lane = head (lane % NH), warp = 16 keys of the page ----------------
     pdl_wait();
     const uint32_t lane_bits = (uint32_t)(warp * 32) << 16;
-    const int row = tid;                                 // the key of the page, for warps 0 and 1
-    float m_ref = -INFINITY;                             // lane h: the reference maximum of head h % NH (base 2), alike in all warps
-    float l[NH];
+    const int hl = lane % NH;
+    if (!wait_bar(q_full, 0, abort_flag)) { ok = false; *abort_flag = 1; }
+    for (int c0 = 0; c0 < p.qcols; c0 += 16) {           // 32 numbers of the head at a time: four 16-byte chunks of its row
+      uint32_t w[16];
 #pragma unroll
-    for (int h = 0; h < NH; ++h) l[h] = 0.f;
+      for (int c = 0; c < 4; ++c) {
+        const int k8 = c0 / 4 + c;                       // chunk of eight numbers
+        const uint4 v = *reinterpret_cast<const uint4*>(q_s + (k8 >> 3) * QBOX + hl * 128 + (((k8 & 7) ^ (hl & 7)) << 4));
+        w[4 * c] = v.x; w[4 * c + 1] = v.y; w[4 * c + 2] = v.z; w[4 * c + 3] = v.w;
+      }
+      tmem_st16_issue(tmem + lane_bits + c0, w);
+    }
+    tmem_st_wait();
+    tc_fence_before();
+    mbar_arrive(q_moved);
+    float m_ref = -INFINITY, l = 0.f;                    // the head's reference maximum (base 2), alike in all warps; this thread's sum
     for (int it = 0; it < n_tiles; ++it) {
-      float sc[NH];
-      if (warp < 2) {
-        const int pg = iert_walk_page(walk, t_lo + it), j = pg * BK + row;
-        const int page = kv.page_table[(size_t)slot * kv.table_width + iert_table_entry(kv, pg)];
-        const bool vis = page >= 0 && page < kv.n_pages && j <= pos && (j >= walk.j_min || j < kv.keep);
-        if (!wait_bar(&s_full[it & 1], (it >> 1) & 1, abort_flag)) ok = false;
-        tc_fence_after();
-        uint32_t raw[NH];
+      const int pg = iert_walk_page(walk, t_lo + it), j0 = pg * BK;
+      const int page = kv.page_table[(size_t)slot * kv.table_width + iert_table_entry(kv, pg)];
+      const bool page_ok = page >= 0 && page < kv.n_pages;
+      const bool partial = !page_ok || j0 + BK - 1 > pos || j0 < walk.j_min;      // some row of the page may not count
+      auto counts = [&](int r) { return page_ok && j0 + r <= pos && (j0 + r >= walk.j_min || j0 + r < kv.keep); };
+      if (!wait_bar(s_full, it & 1, abort_flag)) { ok = false; *abort_flag = 1; }
+      tc_fence_after();
+      float sc[16];
+      tmem_ld16(tmem + lane_bits + s_col + 16 * warp, sc);
+      tc_fence_before();
+      mbar_arrive(s_empty);
 #pragma unroll
-        for (int c = 0; c < NH; c += 16) tmem_ld16_issue(tmem + lane_bits + (it & 1) * NH + c, raw + c);
-        tmem_ld_wait();
-        float mx[NH];
+      for (int c = 0; c < 16; ++c) sc[c] *= p.scale_log2e;
+      if (partial) {
 #pragma unroll
-        for (int h = 0; h < NH; ++h) mx[h] = sc[h] = vis ? __uint_as_float(raw[h]) * p.scale_log2e : -INFINITY;
-        if (!vis) {
+        for (int c = 0; c < 16; ++c) if (!counts(16 * warp + c)) sc[c] = -INFINITY;
+        const int row = tid >> 1;
+        if (!counts(row)) {                              // two threads a row, every other box each
           uint8_t* line = c_s + (it % p.stages) * p.nbox * BOX + row * 128;
-          for (int x = 0; x < p.nbox; ++x)
+          for (int x = tid & 1; x < p.nbox; x += 2)
 #pragma unroll
             for (int c = 0; c < 8; ++c) *reinterpret_cast<uint4*>(line + x * BOX + c * 16) = make_uint4(0u, 0u, 0u, 0u);
         }
-        __syncwarp();
-        const float top = reduce_columns<NH, true>(mx, lane);
-        if (lane < NH) wmax[((it & 1) * 2 + warp) * NH + lane] = top;
-        if (!ok) *abort_flag = 1;
       }
+      float top = sc[0];
+#pragma unroll
+      for (int c = 1; c < 16; ++c) top = fmaxf(top, sc[c]);
+      float* wm = wmax + (it & 1) * 4 * 32;
+      wm[warp * 32 + lane] = top;
       if (tid == 0) stop[it & 1] = *abort_flag;
       soft_sync();
       if (stop[it & 1]) { ok = false; break; }           // all four warps leave at the same barrier
-      const int hl = lane % NH;
-      const float tm = fmaxf(wmax[(it & 1) * 2 * NH + hl], wmax[((it & 1) * 2 + 1) * NH + hl]);
+      const float tm = fmaxf(fmaxf(wm[lane], wm[32 + lane]), fmaxf(wm[64 + lane], wm[96 + lane]));
       const bool grow = tm > m_ref + 8.0f || (m_ref == -INFINITY && tm != -INFINITY);
       if (__any_sync(0xffffffffu, grow)) {               // the same in all four warps
         const float m_new = grow ? tm : m_ref;
         const float alpha = !grow ? 1.f : (m_ref == -INFINITY ? 0.f : ex2(m_ref - m_new));
         m_ref = m_new;
-#pragma unroll
-        for (int h = 0; h < NH; ++h) l[h] *= __shfl_sync(0xffffffffu, alpha, h);
+        l *= alpha;
         if (it > 0) {
           if (!wait_bar(&pv_done[(it - 1) & 1], ((it - 1) >> 1) & 1, abort_flag)) { ok = false; *abort_flag = 1; }
+          __syncwarp();
           tc_fence_after();
           for (int m = 0; m < p.mblocks; ++m)
 #pragma unroll
@@ -282,34 +284,36 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
             }
         }
       }
-      if (warp < 2) {
-        // probabilities: head h is row h of the operand, key `row` its column; the buffer was last read by the sum of page
-        // it - 2, which had finished before the scores of page `it` were committed
-        uint8_t* pb = p_s + (it & 1) * PBUF + (row & 7) * 2;
-        const float neg = m_ref == -INFINITY ? 0.f : -m_ref;
+      // probabilities: head h is row h of the operand, the warp's keys are two 16-byte chunks of it; the buffer was last
+      // read by the sum of page it - 2, which had finished before the scores of page `it` were committed
+      const float neg = m_ref == -INFINITY ? 0.f : -m_ref;
+      uint4 w2[2];
+      __nv_bfloat162* wp = reinterpret_cast<__nv_bfloat162*>(w2);
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
-          const float pr = ex2(sc[h] + __shfl_sync(0xffffffffu, neg, h));
-          l[h] += pr;
-          *reinterpret_cast<__nv_bfloat16*>(pb + h * 128 + (((row >> 3) ^ (h & 7)) << 4)) = __float2bfloat16_rn(pr);
-        }
-        fence_proxy_async_smem();                        // the probabilities, and rows that were cleared, reach the tensor core
+      for (int c = 0; c < 8; ++c) {
+        const float pa = ex2(sc[2 * c] + neg), pb = ex2(sc[2 * c + 1] + neg);
+        l += pa + pb;
+        wp[c] = __floats2bfloat162_rn(pa, pb);
       }
+      if (lane < NH) {
+        uint8_t* pb = p_s + (it & 1) * PBUF + hl * 128;
+        *reinterpret_cast<uint4*>(pb + (((2 * warp) ^ (hl & 7)) << 4)) = w2[0];
+        *reinterpret_cast<uint4*>(pb + (((2 * warp + 1) ^ (hl & 7)) << 4)) = w2[1];
+      }
+      fence_proxy_async_smem();                          // the probabilities, and rows that were cleared, reach the tensor core
       tc_fence_before();
       mbar_arrive(&p_ready[it & 1]);
     }
     if (ok && !wait_bar(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, abort_flag)) ok = false;
-    __syncwarp();
-    const float lw = reduce_columns<NH, false>(l, lane);     // (warps 2 and 3 hold zeros)
-    if (ok && warp == 1 && lane < NH) wsum[lane] = lw;
     if (!ok) *abort_flag = 1;
+    wsum[warp * 32 + lane] = l;
     soft_sync();                                         // every warp has left the loop and said how
     if (tid == 0) stop[0] = *abort_flag;
     soft_sync();
     const bool good = stop[0] == 0;                      // an aborted run leaves an empty partial
     if (warp == 0 && lane < NH) {
       p.part_m[part_row0 + lane] = good && m_ref != -INFINITY ? m_ref * 0.6931471805599453f : -INFINITY;
-      p.part_l[part_row0 + lane] = good ? lw + wsum[lane] : 0.f;
+      p.part_l[part_row0 + lane] = good ? (wsum[lane] + wsum[32 + lane]) + (wsum[64 + lane] + wsum[96 + lane]) : 0.f;
     }
     if (good) {
       tc_fence_after();
@@ -349,15 +353,13 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
   }
 }
 
-size_t fixed_smem(int nh, int nbox) {
+size_t fixed_smem(int nh) {
   const size_t pbuf = (size_t)nh * 128;
-  return (size_t)nbox * nh * 128 + (2 * pbuf > (size_t)BOX ? 2 * pbuf : (size_t)BOX) + (4 * nh + nh) * sizeof(float) +
-         (2 + 2 * MAX_STAGES + 6) * sizeof(uint64_t) + 64;
+  return (2 * pbuf > (size_t)BOX ? 2 * pbuf : (size_t)BOX) + 12 * 32 * sizeof(float) + (9 + 2 * MAX_STAGES) * sizeof(uint64_t) + 32;
 }
 int stages_for(int nh, int width) {
   const int nbox = (width + 63) / 64;
-  const size_t room = 227 * 1024 - fixed_smem(nh, nbox);
-  const int n = (int)(room / ((size_t)nbox * BOX));
+  const int n = (int)((227 * 1024 - fixed_smem(nh)) / ((size_t)nbox * BOX));
   return n > MAX_STAGES ? MAX_STAGES : n;
 }
 
@@ -383,14 +385,14 @@ int launch_latent_decode_umma(const void* qa, const IertBatchView* batch, const 
     return IERT_BAD_ARGUMENT;
   LatentUmmaParams p;
   p.Hpad = Hpad; p.H = H; p.rank = rank;
-  p.nbox = (width + 63) / 64; p.ksteps = (width + 15) / 16; p.mblocks = (rank + 127) / 128;
+  p.nbox = (width + 63) / 64; p.ksteps = (width + 15) / 16; p.qcols = (p.ksteps * 8 + 15) / 16 * 16; p.mblocks = (rank + 127) / 128;
   p.splits = splits; p.stages = stages_for(nh, width);
-  const int cols = 2 * nh + p.mblocks * nh;
+  const int cols = p.qcols + BK + p.mblocks * nh;       // at most 320 + 64 + 128
   p.tmem_cols = 32;
   while ((int)p.tmem_cols < cols) p.tmem_cols *= 2;
   p.scale_log2e = scale * 1.4426950408889634f;
   p.part_m = part_m; p.part_l = part_l; p.part_acc = part_acc; p.err = err;
-  const size_t smem = fixed_smem(nh, p.nbox) + (size_t)p.stages * p.nbox * BOX;
+  const size_t smem = fixed_smem(nh) + (size_t)p.stages * p.nbox * BOX;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(latent_decode_umma_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
