@@ -35,10 +35,11 @@ constexpr int BK = 64;                         // keys per page
 constexpr int BOX = BK * 128;                  // 64 rows x 64 columns of bf16
 constexpr int THREADS = 192, SOFT = 128;
 constexpr uint32_t WAIT_LIMIT = 1u << 22;
+constexpr uint32_t POLL_LIMIT = 1u << 25;      // polls that do not suspend the thread: about as long a wait
 constexpr int MAX_STAGES = 4;
 
 struct LatentUmmaParams {
-  int Hpad, H, rank, nbox, ksteps, qcols, mblocks, splits, stages;
+  int Hpad, H, rank, nbox, qcols, mblocks, splits, stages;
   uint32_t tmem_cols;
   float scale_log2e;
   float* part_m;
@@ -58,6 +59,31 @@ __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+// The MMAs and commits of a whole converged warp of which one lane acts (`leader` != 0): the operands stay warp-uniform,
+// which is what lets one instruction follow another without moving them between register files first.
+__device__ __forceinline__ uint32_t elect_leader() {
+  uint32_t l;
+  asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(l));
+  return l;
+}
+__device__ __forceinline__ void mma_ts(uint32_t leader, uint32_t d, uint32_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %4, 0;\n\tsetp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+      ::"r"(d), "r"(a), "l"(b), "r"(idesc), "r"(accumulate), "r"(leader) : "memory");
+}
+__device__ __forceinline__ void mma_ss(uint32_t leader, uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.b32 p, %4, 0;\n\tsetp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate), "r"(leader) : "memory");
+}
+__device__ __forceinline__ void mma_commit(uint32_t leader, uint64_t* bar) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
+      ::"r"(smem_addr(bar)), "r"(leader) : "memory");
 }
 __device__ __forceinline__ void soft_sync() { asm volatile("bar.sync 1, %0;" ::"n"(SOFT) : "memory"); }
 
@@ -89,7 +115,8 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
   volatile int* stop = armed + 1;                        // [2]: the flag as warp 0 saw it in front of a barrier, so that all agree
 
   const int s = blockIdx.x, split = blockIdx.y, rows0 = blockIdx.z * NH;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int warp = __shfl_sync(0xffffffffu, tid >> 5, 0);          // known to be the same for the whole warp
   const int slot = b.slot_ids[s];
   if (slot < 0) { pdl_wait(); return; }
   const int pos = b.pos0[s];                             // one token per sequence: its own row is in the cache
@@ -168,62 +195,80 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
       *armed = asked;
     }
   } else if (warp == 5) {
-    // ---------------- MMA issuer ----------------
-    if (lane == 0) {
-      constexpr uint32_t IDESC_S = instr_desc_bf16(128, BK);
-      constexpr uint32_t IDESC_L = instr_desc_bf16_a_mn(128, NH);
-      auto scores = [&](int it) {                        // S = Qa C_it^T (the page has landed, the scores before are read)
-        tc_fence_after();
-        const uint32_t cb = smem_addr(c_s + (it % p.stages) * p.nbox * BOX);
-        for (int ks = 0; ks < p.ksteps; ++ks)
-          umma_bf16_a_tmem(tmem + s_col, tmem + ks * 8, smem_desc_k128(cb + (ks / 4) * BOX + (ks % 4) * 32), IDESC_S, ks > 0 ? 1u : 0u);
-        umma_commit(s_full);
-      };
-      ok = wait_bar(q_moved, 0, abort_flag) && wait_bar(&c_full[0], 0, abort_flag);
-      if (ok) scores(0);
-      for (int it = 0; ok && it < n_tiles; ++it) {
-        const int st = it % p.stages, nx = it + 1, sn = nx % p.stages;
-        bool next_done = nx >= n_tiles, ready = false;
-        for (uint32_t i = 0; i < WAIT_LIMIT && !ready; ++i) {
-          if (!next_done && mbar_try_wait(s_empty, it & 1) && mbar_try_wait(&c_full[sn], (nx / p.stages) & 1)) {
-            scores(nx);
-            next_done = true;
-          }
-          ready = mbar_try_wait(&p_ready[it & 1], (it >> 1) & 1);
-          if ((i & 255u) == 255u && *abort_flag) break;
-        }
-        if (!ready) { ok = false; break; }
-        tc_fence_after();
-        const uint32_t cb = smem_addr(c_s + st * p.nbox * BOX), pb = smem_addr(p_s + (it & 1) * PBUF);
-        for (int m = 0; m < p.mblocks; ++m)
+    // ---------------- MMA issuer (the whole warp, one lane of it acting) ----------------
+    constexpr uint32_t IDESC_S = instr_desc_bf16(128, BK);
+    constexpr uint32_t IDESC_L = instr_desc_bf16_a_mn(128, NH);
+    const uint32_t leader = elect_leader();
+    const uint32_t c_base = smem_addr(c_s), stage_bytes = p.nbox * BOX;
+    auto scores = [&](int st) {                          // S = Qa C^T (the page in stage st has landed, the scores before are read)
+      tc_fence_after();
+      uint64_t cd = smem_desc_k128(c_base + st * stage_bytes);
+      uint32_t qa = tmem;
+      mma_ts(leader, tmem + s_col, qa, cd, IDESC_S, 0u);                           // columns beyond `width` are zeros
 #pragma unroll
-          for (int kk = 0; kk < BK / 16; ++kk)
-            umma_bf16(tmem + l_col + m * NH, smem_desc_mn128(cb + 2 * m * BOX + kk * 16 * 128, BOX), smem_desc_k128(pb + kk * 32),
-                      IDESC_L, (it > 0 || kk > 0) ? 1u : 0u);
-        umma_commit(&pv_done[it & 1]);
-        umma_commit(&c_empty[st]);
-        if (!next_done) {
-          if (!wait_bar(s_empty, it & 1, abort_flag) || !wait_bar(&c_full[sn], (nx / p.stages) & 1, abort_flag)) { ok = false; break; }
-          scores(nx);
-        }
+      for (int ks = 1; ks < 4; ++ks) mma_ts(leader, tmem + s_col, qa + ks * 8, cd + ks * 2, IDESC_S, 1u);
+      for (int x = 1; x < p.nbox; ++x) {
+        cd += BOX >> 4;
+        qa += 32;
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) mma_ts(leader, tmem + s_col, qa + ks * 8, cd + ks * 2, IDESC_S, 1u);
       }
-      umma_commit(drained);
+      mma_commit(leader, s_full);
+    };
+    // a wait of the whole warp: what one lane sees, all act on
+    auto warp_wait = [&](uint64_t* bar, uint32_t parity) { return __all_sync(0xffffffffu, wait_bar(bar, parity, abort_flag)) != 0; };
+    ok = warp_wait(q_moved, 0) && warp_wait(&c_full[0], 0);
+    if (ok) scores(0);
+    int st = 0, sn = 1 % p.stages;                       // the stages of page `it` and of the next one, and the next one's phase
+    uint32_t ph = p.stages == 1 ? 1u : 0u;
+    for (int it = 0; ok && it < n_tiles; ++it) {
+      bool next_done = it + 1 >= n_tiles, ready = false;
+      for (uint32_t i = 0; i < POLL_LIMIT && !ready; ++i) {
+        if (!next_done && __all_sync(0xffffffffu, mbar_test(s_empty, it & 1) && mbar_test(&c_full[sn], ph))) {
+          scores(sn);
+          next_done = true;
+        }
+        ready = __all_sync(0xffffffffu, mbar_test(&p_ready[it & 1], (it >> 1) & 1));
+        if ((i & 255u) == 255u && __any_sync(0xffffffffu, *abort_flag != 0)) break;
+      }
+      if (!ready) { ok = false; break; }
+      tc_fence_after();
+      uint64_t cd = smem_desc_mn128(c_base + st * stage_bytes, BOX);
+      const uint64_t pd = smem_desc_k128(smem_addr(p_s) + (it & 1) * PBUF);
+      const uint32_t again = it > 0 ? 1u : 0u;
+      uint32_t d = tmem + l_col;
+      for (int m = 0; m < p.mblocks; ++m) {
+        mma_ss(leader, d, cd, pd, IDESC_L, again);
+#pragma unroll
+        for (int kk = 1; kk < BK / 16; ++kk) mma_ss(leader, d, cd + kk * (16 * 128 >> 4), pd + kk * 2, IDESC_L, 1u);
+        cd += 2 * BOX >> 4;
+        d += NH;
+      }
+      mma_commit(leader, &pv_done[it & 1]);
+      mma_commit(leader, &c_empty[st]);
+      if (!next_done) {
+        if (!warp_wait(s_empty, it & 1) || !warp_wait(&c_full[sn], ph)) { ok = false; break; }
+        scores(sn);
+      }
+      st = sn;
+      if (++sn == p.stages) { sn = 0; ph ^= 1u; }
     }
+    mma_commit(leader, drained);
   } else {
     // ---------------- softmax: lane = head (lane % NH), warp = 16 keys of the page ----------------
     pdl_wait();
     const uint32_t lane_bits = (uint32_t)(warp * 32) << 16;
     const int hl = lane % NH;
     if (!wait_bar(q_full, 0, abort_flag)) { ok = false; *abort_flag = 1; }
-    for (int c0 = 0; c0 < p.qcols; c0 += 16) {           // 32 numbers of the head at a time: four 16-byte chunks of its row
-      uint32_t w[16];
+    for (int x = 0; x < p.nbox; ++x) {                   // 64 numbers of the head at a time: eight 16-byte chunks of its row
+      uint32_t w[32];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int k8 = c0 / 4 + c;                       // chunk of eight numbers
-        const uint4 v = *reinterpret_cast<const uint4*>(q_s + (k8 >> 3) * QBOX + hl * 128 + (((k8 & 7) ^ (hl & 7)) << 4));
+      for (int c = 0; c < 8; ++c) {
+        const uint4 v = *reinterpret_cast<const uint4*>(q_s + x * QBOX + hl * 128 + ((c ^ (hl & 7)) << 4));
         w[4 * c] = v.x; w[4 * c + 1] = v.y; w[4 * c + 2] = v.z; w[4 * c + 3] = v.w;
       }
-      tmem_st16_issue(tmem + lane_bits + c0, w);
+      tmem_st16_issue(tmem + lane_bits + x * 32, w);
+      tmem_st16_issue(tmem + lane_bits + x * 32 + 16, w + 16);
     }
     tmem_st_wait();
     tc_fence_before();
@@ -319,13 +364,14 @@ latent_decode_umma_kernel(const __grid_constant__ CUtensorMap map_c, const __gri
       tc_fence_after();
       for (int m = 0; m < p.mblocks; ++m) {
         const int r = m * 128 + tid;
+        float* dst = p.part_acc + part_row0 * p.rank + r;
 #pragma unroll
         for (int c = 0; c < NH; c += 16) {
           float o[16];
           tmem_ld16(tmem + lane_bits + l_col + m * NH + c, o);
 #pragma unroll
           for (int e = 0; e < 16; ++e)
-            if (r < p.rank && rows0 + c + e < p.H) p.part_acc[(part_row0 + c + e) * p.rank + r] = o[e];
+            if (r < p.rank && rows0 + c + e < p.H) dst[(size_t)(c + e) * p.rank] = o[e];
         }
       }
     }
@@ -385,7 +431,7 @@ int launch_latent_decode_umma(const void* qa, const IertBatchView* batch, const 
     return IERT_BAD_ARGUMENT;
   LatentUmmaParams p;
   p.Hpad = Hpad; p.H = H; p.rank = rank;
-  p.nbox = (width + 63) / 64; p.ksteps = (width + 15) / 16; p.qcols = (p.ksteps * 8 + 15) / 16 * 16; p.mblocks = (rank + 127) / 128;
+  p.nbox = (width + 63) / 64; p.qcols = p.nbox * 32; p.mblocks = (rank + 127) / 128;
   p.splits = splits; p.stages = stages_for(nh, width);
   const int cols = p.qcols + BK + p.mblocks * nh;       // at most 320 + 64 + 128
   p.tmem_cols = 32;
