@@ -351,6 +351,76 @@ latent_prep_kernel(LatentPrep a, IertBatchView b, IertKvView kv, int* __restrict
   }
 }
 
+// The same without queries, a warp per row (the key/value row of a token, or its query latent): the row stays in
+// registers, 16-byte accesses, no barrier.  NV groups of four per lane; rank, q_rank, rank + R and the row strides are
+// multiples of 4.
+template <typename T, int NV>
+__global__ void latent_rows_kernel(LatentPrep a, IertBatchView b, IertKvView kv, int* __restrict__ err) {
+  pdl_launch_dependents();
+  const int pieces = a.dq ? 2 : 1, warps = blockDim.x >> 5, lane = threadIdx.x & 31;
+  const int item = blockIdx.x * warps + (threadIdx.x >> 5);
+  const int t = item / pieces;
+  if (t >= b.n_tokens) { pdl_wait(); return; }
+  const bool latent_q = a.dq && item % 2 == 1;
+  const int n = latent_q ? a.q_rank : a.rank, R = a.R, half = R / 2;
+  const int s = sequence_of_token(b, t);
+  const int slot = s >= 0 ? b.slot_ids[s] : -1;
+  const float* w = latent_q ? a.wq : a.wkv;
+  T* out = latent_q ? (T*)a.cq + (size_t)t * a.q_rank : (T*)a.c_ext + (size_t)t * (a.rank + R);
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (slot < 0) {                        // padding: rows of zeros, nothing stored
+    pdl_wait();
+    for (int i = 4 * lane; i < (latent_q ? n : n + R); i += 128) latent_put4(out + i, zero);
+    if (a.glog && !latent_q) for (int i = lane; i < a.H; i += 32) a.gate_out[(size_t)t * a.H + i] = 0.f;
+    return;
+  }
+  const int pos = b.pos0[s] + (t - b.cu_q[s]);
+  T* dst = nullptr;
+  if (!latent_q && a.store && iert_stays_cached(kv, pos, b.pos0[s] + (b.cu_q[s + 1] - b.cu_q[s]))) {
+    const long long off = kv_row_offset(kv, slot, pos, 0, err);
+    if (off >= 0) dst = (T*)kv.k + off;
+  }
+  pdl_wait();
+  const float* x = latent_q ? a.dq + (size_t)t * a.ld_dq : a.down + (size_t)t * a.ld_down;
+  float4 v[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    v[k] = i < n ? *reinterpret_cast<const float4*>(x + i) : zero;
+    ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+  }
+  const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    if (i < n) {
+      const float4 g = *reinterpret_cast<const float4*>(w + i);
+      const float4 o = make_float4(v[k].x * r * g.x, v[k].y * r * g.y, v[k].z * r * g.z, v[k].w * r * g.w);
+      latent_put4(out + i, o);
+      if (dst) latent_put4(dst + i, o);
+    }
+  }
+  if (latent_q) return;
+  const float* kr = x + a.rank;
+  for (int k = lane; k < half; k += 32) {
+    const int i0 = a.pairing == IERT_PAIR_INTERLEAVED ? 2 * k : k, i1 = a.pairing == IERT_PAIR_INTERLEAVED ? 2 * k + 1 : k + half;
+    const float p = kr[i0], q = kr[i1];
+    float sn, co;
+    sincosf((float)pos * a.inv_freq[k], &sn, &co);
+    sn *= a.rot_mul;
+    co *= a.rot_mul;
+    const T o0 = from_f32<T>(p * co - q * sn), o1 = from_f32<T>(q * co + p * sn);
+    out[a.rank + i0] = o0;
+    out[a.rank + i1] = o1;
+    if (dst) { dst[a.rank + i0] = o0; dst[a.rank + i1] = o1; }
+  }
+  if (a.glog) {
+    const float* g = a.glog + (size_t)t * a.ld_glog;
+    for (int i = lane; i < a.H; i += 32) a.gate_out[(size_t)t * a.H + i] = a.out_scale / (1.0f + expf(-g[i]));
+  }
+}
+
 // out[t, h, :V] = attn[t, h, :V] * gate[t, h]: drops the padding of heads of `head` numbers and applies the gate.
 template <typename T>
 __global__ void head_gate_mul_kernel(const T* __restrict__ attn, int head, T* __restrict__ out, int V, int H,
@@ -468,6 +538,19 @@ IERT_API int iert_latent_prep(const float* q, long long ldq_in, const float* dow
   const int elt = dtype == IERT_F32 ? 4 : 2;
   const bool vec = q && D % 4 == 0 && (R / 2) % 4 == 0 && q_head % 4 == 0 && ldq % 4 == 0 && ldq_in % 4 == 0 && ((uintptr_t)q & 15) == 0 &&
                    ((uintptr_t)q_out % (4 * elt)) == 0;
+  const int longest = dq && q_rank > rank ? q_rank : rank;
+  const bool rows = !q && down && longest <= 2048 && rank % 4 == 0 && (rank + R) % 4 == 0 && ld_down % 4 == 0 && ((uintptr_t)down & 15) == 0 &&
+                    ((uintptr_t)wkv & 15) == 0 && ((uintptr_t)c_ext & 15) == 0 && (!store || ((uintptr_t)kv->k & 15) == 0) &&
+                    (!dq || (q_rank % 4 == 0 && ld_dq % 4 == 0 && ((uintptr_t)dq & 15) == 0 && ((uintptr_t)wq & 15) == 0 && ((uintptr_t)cq & 15) == 0));
+  if (rows) {
+    const int items = batch->n_tokens * (dq ? 2 : 1), threads = batch->n_tokens >= 256 ? 128 : 32, warps = threads / 32;
+#define ROWS(T, NV) launch_dep(latent_rows_kernel<T, NV>, dim3((items + warps - 1) / warps), dim3(threads), 0, stream, a, *batch, *kv, err)
+    if (dtype == IERT_F32) { if (longest <= 512) ROWS(float, 4); else ROWS(float, 16); }
+    else if (dtype == IERT_BF16) { if (longest <= 512) ROWS(__nv_bfloat16, 4); else ROWS(__nv_bfloat16, 16); }
+    else return IERT_BAD_ARGUMENT;
+#undef ROWS
+    return iert_check_launch("latent_prep");
+  }
 #define GO(T)                                                                                                                        \
   do {                                                                                                                               \
     if (vec) launch_dep(latent_prep_kernel<T, true>, dim3(batch->n_tokens), dim3(256), R * sizeof(float), stream, a, *batch, *kv, err); \
