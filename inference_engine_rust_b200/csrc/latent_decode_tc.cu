@@ -44,6 +44,12 @@ __device__ __forceinline__ uint32_t lds32(const __nv_bfloat16* p) { return *rein
 // weights) times four groups along d, added through shared memory in a fixed order.
 constexpr int ABSORB_THREADS = 256;
 
+// Asks for `bytes` bytes of weights to be brought into the L2 while the block still waits for the kernel in front.
+__device__ __forceinline__ void fetch_ahead(const void* p, size_t bytes) {
+  for (size_t i = (size_t)threadIdx.x * 128; i < bytes; i += (size_t)blockDim.x * 128)
+    asm volatile("prefetch.global.L2 [%0];" ::"l"((const char*)p + i));
+}
+
 // TQ float: q is the projection as it stands, and the R last numbers of a head are turned here (inv_freq, rot_mul, pairing).
 template <typename TQ, int TT>
 __global__ void __launch_bounds__(ABSORB_THREADS)
@@ -55,6 +61,7 @@ latent_absorb_q_kernel(const TQ* __restrict__ q, long long ldq, const __nv_bfloa
   float* part = sm_q + TT * D;          // [4][TT][rank]
   pdl_launch_dependents();
   const int t0 = blockIdx.x * TT, h = blockIdx.y, n_t = min(TT, b.n_tokens - t0);
+  if (blockIdx.x == 0 && h < H) fetch_ahead(w_uk + (size_t)h * D * rank, (size_t)D * rank * 2);
   pdl_wait();
   if (h >= H) {                         // heads that only fill the MMA tile
     for (int i = threadIdx.x; i < n_t * (rank + R); i += blockDim.x)
@@ -320,6 +327,9 @@ latent_decode_merge_kernel(const float* __restrict__ part_m, const float* __rest
   pdl_launch_dependents();
   const int t0 = blockIdx.x * TT, h = blockIdx.y, n_t = min(TT, b.n_seqs - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  // this block's rows of W_uv: several blocks share a head's (each merges the runs for itself)
+  const int per_z = (V + gridDim.z - 1) / gridDim.z, e_lo = blockIdx.z * per_z, e_hi = min(V, e_lo + per_z);
+  if (blockIdx.x == 0 && e_lo < e_hi) fetch_ahead(w_uv + ((size_t)h * V + e_lo) * rank, (size_t)(e_hi - e_lo) * rank * sizeof(T));
   pdl_wait();
   for (int t = warp; t < TT; t += MERGE_THREADS / 32) {          // splits <= 64: two runs per lane
     const bool live = t < n_t && b.slot_ids[t0 + t] >= 0;        // a padding sequence: weights of zero
@@ -345,27 +355,34 @@ latent_decode_merge_kernel(const float* __restrict__ part_m, const float* __rest
     for (int k = 0; k < 2; ++k) wgt[t * 64 + lane + 32 * k] = lane + 32 * k < splits ? w[k] * inv : 0.f;
   }
   __syncthreads();
-  // the runs' partial sums, eight loads in flight per thread; an empty run's row (weight 0) is never read
-  for (int j = threadIdx.x; j < TT * rank; j += MERGE_THREADS) {
-    const int t = j / rank, r = j - t * rank;
+  // the runs' partial sums, four numbers per thread, four runs' loads in flight; an empty run's row (weight 0) is never read
+  const int r4 = rank >> 2;
+  for (int j = threadIdx.x; j < TT * r4; j += MERGE_THREADS) {
+    const int t = j / r4, r = 4 * (j - t * r4);
     const float* wt = wgt + t * 64;
-    float a = 0.f;
-    for (int i0 = 0; i0 < splits; i0 += 8) {
-      float v[8];
+    const float* src = part_acc + (((size_t)(t0 + t) * splits) * Hpad + h) * rank + r;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i0 = 0; i0 < splits; i0 += 4) {
+      float4 v[4];
+      float w[4];
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const int i = i0 + k;
-        v[k] = (i < splits && wt[i] != 0.f) ? part_acc[(((size_t)(t0 + t) * splits + i) * Hpad + h) * rank + r] : 0.f;
+      for (int k = 0; k < 4; ++k) {
+        w[k] = wt[(i0 + k) & 63];                       // zero beyond the last run
+        v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (w[k] != 0.f) v[k] = *reinterpret_cast<const float4*>(src + (size_t)(i0 + k) * Hpad * rank);
       }
 #pragma unroll
-      for (int k = 0; k < 8; ++k) a = fmaf(wt[(i0 + k) & 63], v[k], a);
+      for (int k = 0; k < 4; ++k) {
+        a.x = fmaf(w[k], v[k].x, a.x); a.y = fmaf(w[k], v[k].y, a.y);
+        a.z = fmaf(w[k], v[k].z, a.z); a.w = fmaf(w[k], v[k].w, a.w);
+      }
     }
-    lat[j] = a;
+    *reinterpret_cast<float4*>(lat + 4 * j) = a;
   }
   __syncthreads();
   // W_uv: rank is a multiple of 8, 16-byte loads of eight weights; the loads of ROWS rows are issued before the first is used
   constexpr int ROWS = TT > 2 ? 4 : 8;
-  for (int e0 = warp * ROWS; e0 < V; e0 += (MERGE_THREADS / 32) * ROWS) {
+  for (int e0 = e_lo + warp * ROWS; e0 < e_hi; e0 += (MERGE_THREADS / 32) * ROWS) {
     float a[ROWS][TT];
 #pragma unroll
     for (int k = 0; k < ROWS; ++k)
@@ -375,7 +392,7 @@ latent_decode_merge_kernel(const float* __restrict__ part_m, const float* __rest
       uint4 v[ROWS];
 #pragma unroll
       for (int k = 0; k < ROWS; ++k)
-        v[k] = e0 + k < V ? *reinterpret_cast<const uint4*>(w_uv + ((size_t)h * V + e0 + k) * rank + r) : make_uint4(0u, 0u, 0u, 0u);
+        v[k] = e0 + k < e_hi ? *reinterpret_cast<const uint4*>(w_uv + ((size_t)h * V + e0 + k) * rank + r) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
       for (int t = 0; t < TT; ++t) {
         float x[8];
@@ -398,7 +415,7 @@ latent_decode_merge_kernel(const float* __restrict__ part_m, const float* __rest
 #pragma unroll
       for (int t = 0; t < TT; ++t) {
         const float sum = warp_sum(a[k][t]);
-        if (lane == 0 && e0 + k < V && t < n_t)
+        if (lane == 0 && e0 + k < e_hi && t < n_t)
           out[((size_t)(t0 + t) * H + h) * V + e0 + k] = from_f32<T>(gate ? sum * gate[(size_t)(t0 + t) * H + h] : sum);
       }
   }
@@ -497,7 +514,7 @@ IERT_API int iert_latent_attention_decode_tc(const void* q, int q_f32, long long
     launch_dep(latent_decode_tc_kernel<1>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16*)qa, *batch, *kv, Hpad, R,
                scale, splits, part_m, part_l, part_acc, err);
 #define MERGE(TT)                                                                                                                  \
-  launch_dep(latent_decode_merge_kernel<__nv_bfloat16, TT>, dim3((T + TT - 1) / TT, H), dim3(MERGE_THREADS),                       \
+  launch_dep(latent_decode_merge_kernel<__nv_bfloat16, TT>, dim3((T + TT - 1) / TT, H, V >= 64 && T <= 8 ? 2 : 1), dim3(MERGE_THREADS),                       \
              (size_t)TT * (rank + 64) * sizeof(float), stream, (const float*)part_m, (const float*)part_l, (const float*)part_acc, splits, \
              Hpad, rank, sink, gate, (const __nv_bfloat16*)w_uv, (__nv_bfloat16*)out, *batch, H, V)
   if (tt == 1) MERGE(1);
