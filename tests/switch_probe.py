@@ -3,6 +3,7 @@ the environment when the libraries load): a fixed workload through the engine an
 projection kernel, its results saved with torch.save to the path given as the only argument.
 
   * Tiny A in bfloat16: four prompts of unequal lengths in one step, then eight tokens each;
+  * a Botulorn model of four layers with latent attention (one-token steps over cached rows) likewise;
   * two layers at 7B sizes in bfloat16: a 300-token prompt whole, then three requests batched,
     their last 32 / 5 / 17 tokens one by one (split-K projections, decode attention over
     several pages, a window of 160 that cuts the longest request);
@@ -19,6 +20,7 @@ sys.path.insert(0, os.path.dirname(TESTS))
 sys.path.insert(0, TESTS)
 
 from helpers import TINY_A, prompts_for                                 # noqa: E402
+from test_gpu_botulorn import TENSOR                                    # noqa: E402
 from test_gpu_full_size import CFG, LENGTHS, run_batched_with_tails     # noqa: E402
 
 
@@ -26,17 +28,18 @@ def main(path: str) -> None:
     from inference_engine_rust_b200 import LoadedModel
     from inference_engine_rust_b200.csrc import bindings as B
     out = {}
-    tiny = LoadedModel.random(dict(TINY_A), seed=3, dtype="bfloat16", std=0.1)
-    eng = tiny.session(max_tokens=64 * 8, poison_cache=True).engine
-    prompts = prompts_for(TINY_A, [5, 11, 23, 70], seed=2)
-    slots = [eng.open_sequence() for _ in prompts]
-    rows = [eng.step(list(zip(slots, prompts)), want="all").clone()]
-    g = torch.Generator().manual_seed(1)
-    for _ in range(8):
-        toks = torch.randint(0, TINY_A["vocab_size"], (len(slots),), generator=g).tolist()
-        rows.append(eng.step([(s, [t]) for s, t in zip(slots, toks)], want="last").clone())
-    eng.check_device()
-    out["tiny"] = torch.cat(rows).cpu()
+    for name, cfg, vocab in (("tiny", dict(TINY_A), TINY_A["vocab_size"]), ("latent", TENSOR, TENSOR["vocab"])):
+        tiny = LoadedModel.random(cfg, seed=3, dtype="bfloat16", std=0.1)
+        eng = tiny.session(max_tokens=64 * 8, poison_cache=True).engine
+        prompts = prompts_for({"vocab_size": vocab}, [5, 11, 23, 70], seed=2)
+        slots = [eng.open_sequence() for _ in prompts]
+        rows = [eng.step(list(zip(slots, prompts)), want="all").clone()]
+        g = torch.Generator().manual_seed(1)
+        for _ in range(8):
+            toks = torch.randint(0, vocab, (len(slots),), generator=g).tolist()
+            rows.append(eng.step([(s, [t]) for s, t in zip(slots, toks)], want="last").clone())
+        eng.check_device()
+        out[name] = torch.cat(rows).cpu()
 
     big = LoadedModel.random(CFG, seed=5, dtype="bfloat16", std=0.02, on_device=True)
     g = torch.Generator().manual_seed(3)

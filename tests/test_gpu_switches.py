@@ -34,6 +34,7 @@ SWITCHES = {            # switch -> are the results equal to the bit with it off
     "IERT_DECODE_BALANCE": False,
     "IERT_GEMM_ROWS_MAX": False,        # 0: one-token projections on the tcgen05 kernel with split-K
     "IERT_NORM_AHEAD": False,           # 0: every norm a kernel of its own
+    "IERT_LATENT_UMMA": False,          # 0: one-token latent attention on mma.sync
 }
 
 
