@@ -171,6 +171,39 @@ PRESETS["botulorn-12b-sizes"] = _botulorn(5120, 131072, 40, 32, 8, 128, 128, 409
 PRESETS["botulorn-tiny"] = _botulorn(80, 320, 4, 6, 3, 16, 24, 20, 2, 12, 8, 16, 24, 40, 28, 72, 101, 64)
 
 
+def _gidurax(width, vocab, layers, inner, state, dt_rank, delta_heads, delta_kv, delta_dim, delta_vdim, heads, kv_heads, dim, vdim, ff,
+             experts, identity, top, expert_ff, shared_ff, every, taps=4, loop=None):
+    """A Gidurax configuration whose layers go round selective scan (dense feed-forward), delta rule (experts), attention
+    (dense), attention (experts); `loop` = (start, stop, times)."""
+    mixers = [
+        ("mamba1", {"inner": inner, "state": state, "dt_rank": dt_rank, "conv": taps}),
+        ("delta", {"heads": delta_heads, "kv_heads": delta_kv, "dim": delta_dim, "vdim": delta_vdim, "conv": taps}),
+        ("attention", {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
+                       "q_temp": {"coef": 0.1, "every": every}}),
+    ]
+    mlps = [{"kind": "dense", "ff": ff},
+            {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "identity": identity, "top": top},
+             "shared": {"ff": shared_ff}}]
+    out = []
+    for i in range(layers):
+        kind, mixer = mixers[min(i % 4, 2)]
+        out.append({"type": kind, "mixer": copy.deepcopy(mixer), "mlp": copy.deepcopy(mlps[i % 2])})
+    cfg = {"architecture": "Gidurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+           "residual_mult": 0.5, "layers": out}
+    if loop is not None:
+        cfg["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return cfg
+
+
+# Gidurax at the width, head count, head size and total feed-forward size (14 experts of 896 and a shared one of 1,792 = 14,336) of
+# Mistral 7B (a scan twice as wide as the model with 16 states per channel), and a tiny one that runs anywhere in seconds (value sizes
+# unlike the key sizes, its layers 1 and 2 run three times).
+PRESETS["gidurax-7b-sizes"] = _gidurax(4096, 32000, 32, 8192, 16, 256, 32, 32, 128, 128, 32, 8, 128, 128, 14336, 14, 2, 2, 896, 1792, 4096)
+# the same at the sizes of Mistral NeMo 12B (width 5,120, a vocabulary of 131,072)
+PRESETS["gidurax-12b-sizes"] = _gidurax(5120, 131072, 40, 10240, 16, 320, 32, 32, 128, 128, 32, 8, 128, 128, 14336, 14, 2, 2, 896, 1792, 4096)
+PRESETS["gidurax-tiny"] = _gidurax(80, 320, 5, 112, 12, 20, 6, 3, 32, 24, 6, 2, 16, 24, 136, 5, 3, 3, 40, 24, 16, taps=3, loop=(1, 3, 3))
+
+
 def preset(name: str) -> dict:
     """A copy of the named configuration (a config.json-style dict)."""
     try:

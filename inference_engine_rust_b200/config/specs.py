@@ -53,10 +53,12 @@ class ScheduleEntry:
     """One execution of a layer.  `layer` indexes `ModelSpec.layers`; a layer may be named
     by several entries (shared weights), and each entry that writes a cache has storage of
     its own.  `reads_cache_of` names an EARLIER entry of the schedule (by its position)
-    whose cache this execution reads instead of writing one."""
+    whose cache this execution reads instead of writing one.  `pass_start` t: pass number t of a
+    repeated run of layers starts here; the model's `passes` part changes the residual first."""
 
     layer: int
     reads_cache_of: Optional[int] = None
+    pass_start: Optional[int] = None
 
     @property
     def writes_cache(self) -> bool:
@@ -86,6 +88,8 @@ class ModelSpec:
     # ([tokens, S, hidden], all equal to the embedded row at the start, summed before the final norm);
     # the blocks of such a model take the streams, and the norms need `forward_streams`.
     residual_streams: Optional[int] = None
+    # What runs right before the schedule entries that start a pass: (spec, tensor-name prefix).
+    passes: Optional[Tuple[PartSpec, str]] = None
 
     def validate(self) -> None:
         n = len(self.layers)
@@ -96,6 +100,9 @@ class ModelSpec:
         for pos, e in enumerate(self.schedule):
             if not 0 <= e.layer < n:
                 raise ValueError(f"schedule entry {pos} names layer {e.layer}, the model has {n}")
+            if e.pass_start is not None and (self.passes is None or self.residual_streams is not None):
+                raise ValueError(f"schedule entry {pos} starts a pass, but the model "
+                                 f"{'has no part for that' if self.passes is None else 'keeps its residual as streams'}")
             if e.reads_cache_of is not None:
                 src = e.reads_cache_of
                 if not 0 <= src < pos:

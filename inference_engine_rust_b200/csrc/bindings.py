@@ -62,6 +62,26 @@ class GatedAct(Structure):
     _fields_ = [("g_max", c_float), ("u_max", c_float), ("u_bias", c_float), ("a", c_float), ("b", c_float)]
 
 
+ACT_NONE, ACT_GELU, ACT_SOFTPLUS = 0, 1, 2
+PLAIN_ACTIVATIONS = {"none": ACT_NONE, "gelu": ACT_GELU, "softplus": ACT_SOFTPLUS}     # "gelu": the exact (erf) form
+
+
+class Epilogue(Structure):
+    """Mirror of `IertEpilogue` (common.cuh): v <- act(v + bias[n]) * scale[t, min(n / block_cols, blocks)]."""
+    _fields_ = [("act", c_int), ("bias", c_void_p), ("scale", c_void_p), ("ld_scale", c_longlong), ("blocks", c_int),
+                ("block_cols", c_int)]
+
+
+def epilogue(act: str = "none", bias=None, scale=None, blocks: int = 0, block_cols: int = 1) -> Epilogue:
+    """What a projection does to each output before it stores it: `bias` fp32 [N], an activation by name, and a factor per
+    token and block of columns (`scale` fp32 [tokens, > blocks]: `blocks` blocks of `block_cols` columns, the rest one more)."""
+    if act not in PLAIN_ACTIVATIONS:
+        raise KernelError(f"activation must be one of {sorted(PLAIN_ACTIVATIONS)}, got {act!r}")
+    return Epilogue(act=PLAIN_ACTIVATIONS[act], bias=bias.data_ptr() if bias is not None else None,
+                    scale=scale.data_ptr() if scale is not None else None, ld_scale=scale.stride(0) if scale is not None else 0,
+                    blocks=blocks, block_cols=block_cols)
+
+
 def gated_act(name: str, limit: Optional[float] = None) -> Optional[GatedAct]:
     """The constants of a named gated activation: "silu" (None: the kernels' default), "gelu_tanh" (the tanh form
     of GELU), "clamped_swish" (gate capped at `limit`, up clamped to +-`limit` and shifted by one, sigmoid of
@@ -127,7 +147,8 @@ def _declare(lib) -> None:
         "iert_sample_temperature": [P, c_int, c_int, c_longlong, c_float, c_ulonglong, P, P, P, P, S],
         "iert_uniform_draws": [c_ulonglong, P, P, P, c_int, S],
         "iert_gemm_tc": [P, c_longlong, P, c_longlong, P, c_int, c_longlong, c_int, c_int, c_int, c_int,
-                         P, c_longlong, P, c_int, c_int, c_int, c_int, P, S],
+                         P, c_longlong, P, c_int, c_int, c_int, c_int, POINTER(Epilogue), P, S],
+        "iert_epilogue_rows": [P, c_int, c_longlong, c_int, c_int, POINTER(Epilogue), S],
     }
     LL = c_longlong
     sigs.update({
@@ -154,11 +175,14 @@ def _declare(lib) -> None:
         "iert_router_topk": [P, LL, P, c_int, c_int, c_int, P, P, P, S],
         "iert_moe_scale": [P, c_int, LL, P, c_int, c_int, c_int, P, P, LL, P, c_int, S],
         "iert_router_grouped": [P, LL, LL, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                P, P, P, P, S],
+                                c_int, c_int, P, c_int, P, P, P, P, c_int, LL, P, c_int, S],
         "iert_qkv_prep": [P, LL, P, P, c_int, POINTER(BatchView), POINTER(KvView), c_int, c_int, c_int, P, c_int, c_float, c_int,
-                          P, P, c_float, P, LL, c_float, c_int, P, S],
+                          P, P, c_float, P, LL, c_float, c_float, c_float, c_int, P, S],
         "iert_gate_mul": [P, P, LL, c_int, P, c_int, c_int, c_int, c_int, c_int, S],
-        "iert_add_normed": [P, P, P, P, c_int, c_int, c_int, c_float, S],
+        "iert_add_normed": [P, P, P, P, c_int, c_int, c_int, c_float, P, c_float, S],
+        "iert_rows_begin": [P, P, P, P, P, P, c_int, c_int, c_int, P, c_float, S],
+        "iert_selective_conv": [P, c_int, LL, P, P, P, LL, LL, P, c_int, c_int, POINTER(BatchView), S],
+        "iert_selective_scan": [P, c_int, P, P, LL, P, LL, P, P, P, LL, LL, P, c_int, c_int, c_int, POINTER(BatchView), S],
         "iert_cast_rows": [P, P, P, c_int, LL, S],
         "iert_scale_values": [P, LL, c_float, S],
         "iert_qk_prep": [P, LL, P, c_int, POINTER(BatchView), POINTER(KvView), c_int, P, c_int, c_int, P, P, c_float, c_float,
@@ -175,7 +199,7 @@ def _declare(lib) -> None:
                                        c_int, c_int, P, S]
     lib.iert_gemm_tc_gated.restype = c_int
     lib.iert_gemm_rows.argtypes = [P, c_longlong, P, c_longlong, P, c_int, c_longlong, c_int, c_int, c_int, c_int,
-                                   POINTER(RowScale), POINTER(NormAhead), c_int, c_int, P, S]
+                                   POINTER(RowScale), POINTER(NormAhead), POINTER(Epilogue), c_int, c_int, P, S]
     lib.iert_gemm_rows.restype = c_int
     lib.iert_gemm_tc_scaled.argtypes = [P, c_longlong, P, c_longlong, P, c_int, c_longlong, c_int, c_int, c_int, c_int,
                                         P, c_longlong, P, c_int, POINTER(RowScale), POINTER(NormAhead), c_int, c_int, P, S]
@@ -301,6 +325,12 @@ def gated_act_mul(gu, out, n_tokens: int, inter: int, act: GatedAct, stream) -> 
           "gated_act_mul")
 
 
+def epilogue_rows(z, n_rows: int, ep: Epilogue, stream) -> None:
+    """A projection's epilogue on its stored rows z [T, N], in place."""
+    check(core().iert_epilogue_rows(z.data_ptr(), dtype_code(z.dtype), z.stride(0), n_rows, z.shape[1], byref(ep), stream),
+          "epilogue_rows")
+
+
 def add_into(residual, y, n: int, stream) -> None:
     check(core().iert_add_into(residual.data_ptr(), y.data_ptr(), dtype_code(y.dtype), n, stream),
           "add_into")
@@ -377,15 +407,16 @@ def gemm_tc_set_poll_limit(polls: int) -> None:
 
 
 def gemm_tc(x, w, out, M: int, mode: int, err, stream, force_bt: int = 0, force_splits: int = 0,
-            force_stages: int = 0) -> bool:
-    """out[:M] (=|+=) x[:M] @ w.T on the tensor cores (bf16 operands).  Returns False, having
+            force_stages: int = 0, epilogue: Optional[Epilogue] = None) -> bool:
+    """out[:M] (=|+=) x[:M] @ w.T on the tensor cores (bf16 operands); `epilogue` (plain stores): what is done to the outputs.  Returns False, having
     launched nothing, when the operands do not meet the kernel's alignment rules."""
     N, K = w.shape
     sc = GemmScratch.get(x.device)
     status = core().iert_gemm_tc(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(),
                                  dtype_code(out.dtype), out.stride(0), M, N, K, mode, sc.ws.data_ptr(),
                                  sc.ws.numel(), sc.counters.data_ptr(), sc.counters.numel(), force_bt,
-                                 force_splits, force_stages, err.data_ptr(), stream)
+                                 force_splits, force_stages, byref(epilogue) if epilogue is not None else None, err.data_ptr(),
+                                 stream)
     if status == 1:
         return False
     check(status, "gemm_tc")
@@ -393,7 +424,8 @@ def gemm_tc(x, w, out, M: int, mode: int, err, stream, force_bt: int = 0, force_
 
 
 def gemm_rows(x, w, out, M: int, mode: int, err, stream, scale: Optional[RowScale] = None,
-              ahead: Optional[NormAhead] = None, force_stages: int = 0, w_dynamic: bool = False) -> bool:
+              ahead: Optional[NormAhead] = None, force_stages: int = 0, w_dynamic: bool = False,
+              epilogue: Optional[Epilogue] = None) -> bool:
     """out[:M] (=|+=) x[:M] @ w.T for one-token steps (M <= 32, bf16 operands): 16 weight rows per
     CTA over all of k, no split-K.  `scale`: x is the first half of an RMSNorm and the outputs
     are multiplied by the rows' 1 / rms; `ahead` (with a residual add): the first half of the
@@ -404,7 +436,8 @@ def gemm_rows(x, w, out, M: int, mode: int, err, stream, scale: Optional[RowScal
     status = core().iert_gemm_rows(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(),
                                    dtype_code(out.dtype), out.stride(0), M, N, K, mode,
                                    byref(scale) if scale is not None else None,
-                                   byref(ahead) if ahead is not None else None, force_stages, 1 if w_dynamic else 0,
+                                   byref(ahead) if ahead is not None else None,
+                                   byref(epilogue) if epilogue is not None else None, force_stages, 1 if w_dynamic else 0,
                                    err.data_ptr(), stream)
     if status == 1:
         return False
@@ -817,16 +850,22 @@ ROUTER_GROUP_SCORES = {"max": 0, "top2_sum": 1}
 
 def router_grouped(z, correction, n_tokens: int, E: int, N: int, top: int, groups: int, keep: int, wt, wid, idx, w,
                    stream, by_output: bool = False, score: str = "softmax", group_score: str = "max",
-                   weight_eps: float = 1e-20, weight_scale: float = 1.0) -> None:
+                   weight_eps: float = 1e-20, weight_scale: float = 1.0, renormalize: bool = True, shared_gate: bool = False,
+                   x=None, residual=None) -> None:
     """Scores = softmax over all N router outputs, or each output's sigmoid (the last N - E stand for experts that return
     their input); choice on score + correction inside the `keep` best of `groups` runs of neighbours (a run's score: its
     best choice score, or the sum of its two best); weights = chosen scores over (their sum + weight_eps), times
-    weight_scale.  z: fp32 [T, N], or with `by_output` [N, T] (a row per router output).  wt [T, E] dense, wid [T] the
-    identity experts' share, idx / w [T, top]."""
+    weight_scale (`renormalize` False: chosen scores times weight_scale).  z: fp32 [T, N], or with `by_output` [N, T] (a row
+    per router output).  wt [T, E] dense, wid [T] the identity experts' share, idx / w [T, top].  `shared_gate`: z has one
+    output more, the logit of a gate, whose sigmoid becomes wt[:, E].  `x` [T, H] with `residual` (fp32): the identity
+    experts' share is added, residual[t] += wid[t] x[t]."""
     ldz, lde = (z.stride(1), z.stride(0)) if by_output else (z.stride(0), z.stride(1))
     check(core().iert_router_grouped(z.data_ptr(), ldz, lde, _ptr(correction), n_tokens, E, N, top, groups, keep,
                                      ROUTER_SCORES[score], ROUTER_GROUP_SCORES[group_score], weight_eps, weight_scale,
-                                     wt.data_ptr(), wid.data_ptr(), idx.data_ptr(), w.data_ptr(), stream), "router_grouped")
+                                     1 if renormalize else 0, 1 if shared_gate else 0, wt.data_ptr(), wt.stride(0), wid.data_ptr(),
+                                     idx.data_ptr(), w.data_ptr(), _ptr(x), dtype_code(x.dtype) if x is not None else F32,
+                                     x.stride(0) if x is not None else 0, _ptr(residual),
+                                     residual.shape[-1] if residual is not None else 0, stream), "router_grouped")
 
 
 def moe_scale(act, wt, n_tokens: int, E: int, F: int, stream, wid=None, x=None, residual=None) -> None:
@@ -840,12 +879,20 @@ def moe_scale(act, wt, n_tokens: int, E: int, F: int, stream, wid=None, x=None, 
 # norm on a sublayer's output, keys that double as values, the gated linear recurrence
 
 
-def add_normed(x, y, w, cast, rows: int, eps: float, stream) -> None:
+def add_normed(x, y, w, cast, rows: int, eps: float, stream, w2=None, eps2: float = 0.0) -> None:
     """x[:rows] += y / rms(y) * w (fp32; w with any offset already added); y's rows are cleared; `cast`
-    (optional) receives the new rows in its dtype."""
+    (optional) receives the new rows in its dtype, or with `w2` (fp32) their norm x / rms(x) * w2."""
     check(core().iert_add_normed(x.data_ptr(), y.data_ptr(), w.data_ptr(), _ptr(cast),
-                                 dtype_code(cast.dtype) if cast is not None else F32, rows, x.shape[-1], eps, stream),
-          "add_normed")
+                                 dtype_code(cast.dtype) if cast is not None else F32, rows, x.shape[-1], eps, _ptr(w2),
+                                 eps2, stream), "add_normed")
+
+
+def rows_begin(x, rows: int, stream, *, e=None, step=None, keep=None, y=None, out=None, w2=None, eps2: float = 0.0) -> None:
+    """x[:rows] += e[:rows] + step (each optional; `keep` receives what stood in x); y's rows (optional) are cleared; `out`
+    (optional) receives x / rms(x) * w2 (w2 fp32) of the new rows."""
+    check(core().iert_rows_begin(x.data_ptr(), _ptr(e), _ptr(step), _ptr(keep), _ptr(y), _ptr(out),
+                                 dtype_code(out.dtype) if out is not None else F32, rows, x.shape[-1], _ptr(w2), eps2, stream),
+          "rows_begin")
 
 
 def cast_rows(x, y, cast, rows: int, stream) -> None:
@@ -871,14 +918,16 @@ def qk_prep(proj, qkv, batch: BatchView, kv: KvView, heads: int, inv_freq, rotar
 
 
 def qkv_prep(proj, bias, qkv, batch: BatchView, kv: KvView, heads: int, dim: int, vdim: int, inv_freq, rotary_dim: int,
-             pairing: int, wq, wk, eps: float, store: bool, err, stream, rot_mul: float = 1.0, v_first=None, lam: float = 0.0) -> None:
+             pairing: int, wq, wk, eps: float, store: bool, err, stream, rot_mul: float = 1.0, v_first=None, lam: float = 0.0,
+             temp_coef: float = 0.0, temp_every: float = 0.0) -> None:
     """From the fp32 projection rows that begin with [q | k | v] (+ `bias`) to the packed rows [q' | k' | v'] with every
     head padded with zeros to the cache's head size: per-head weighted RMS norm of q and k (`wq`, `wk` of length `dim`,
     optional), rotation (cosine and sine times `rot_mul`), values mixed with another layer's (v <- (1 - lam) v + lam v_first,
-    `v_first` fp32 rows that may be strided), one rounding, and the cache write of k' and v'."""
+    `v_first` fp32 rows that may be strided), queries times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) at position p
+    (temp_every > 0), one rounding, and the cache write of k' and v'."""
     check(core().iert_qkv_prep(proj.data_ptr(), proj.stride(0), _ptr(bias), qkv.data_ptr(), dtype_code(qkv.dtype), byref(batch),
                                byref(kv), heads, dim, vdim, _ptr(inv_freq), rotary_dim, rot_mul, pairing, _ptr(wq), _ptr(wk), eps,
-                               _ptr(v_first), v_first.stride(0) if v_first is not None else 0, lam,
+                               _ptr(v_first), v_first.stride(0) if v_first is not None else 0, lam, temp_coef, temp_every,
                                1 if store else 0, err.data_ptr(), stream), "qkv_prep")
 
 
@@ -929,3 +978,18 @@ def rglru_scan(A, Bv, proj, by, bx, state, out, out_scale: float, C: int, K: int
     check(core().iert_rglru_scan(A.data_ptr(), Bv.data_ptr(), proj.data_ptr(), proj.stride(0), by.data_ptr(), bx.data_ptr(),
                                  state.data_ptr(), state.stride(0), out.data_ptr(), dtype_code(out.dtype), out_scale, C, K,
                                  max_q_len, _ptr(scratch), byref(batch), stream), "rglru_scan")
+
+
+def selective_conv(x, taps, bias, state, ring_off: int, u, C: int, K: int, batch: BatchView, stream) -> None:
+    """u = silu(causal convolution of x's first C columns + bias); taps fp32 [K, C]; the last inputs live in `state` at ring_off."""
+    check(core().iert_selective_conv(x.data_ptr(), dtype_code(x.dtype), x.stride(0), taps.data_ptr(), bias.data_ptr(), state.data_ptr(),
+                                     state.stride(0), ring_off, u.data_ptr(), C, K, byref(batch), stream), "selective_conv")
+
+
+def selective_scan(u, dt, bc, z, A2, D, state, s_off: int, out, C: int, N: int, one_token: bool, batch: BatchView, stream) -> None:
+    """S[c, n] <- exp(dt A) S + dt u B; out = (sum_n S C + D u) * silu(z) over the step's tokens; `bc`: rows that begin with
+    [B | C], `z`: rows of C numbers (both views that may be strided, in u's dtype), dt fp32 [T, C], A2 = A log2(e) (u fp32: A) fp32 [C, N],
+    S [C, N] per slot in `state` at s_off."""
+    check(core().iert_selective_scan(u.data_ptr(), dtype_code(u.dtype), dt.data_ptr(), bc.data_ptr(), bc.stride(0), z.data_ptr(),
+                                     z.stride(0), A2.data_ptr(), D.data_ptr(), state.data_ptr(), state.stride(0), s_off,
+                                     out.data_ptr(), C, N, 1 if one_token else 0, byref(batch), stream), "selective_scan")

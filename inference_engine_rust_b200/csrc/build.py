@@ -37,6 +37,7 @@ CORE_SOURCES = [
     "gemm_tc.cu", "gemm_rows.cu", "attention_decode.cu",
     "streams_norm.cu", "recurrent_prep.cu", "latent_attention.cu", "latent_decode_tc.cu", "moe.cu",
     "outnorm.cu", "qk_prep.cu", "rglru.cu", "qkv_prep.cu", "layernorm.cu", "embed_pairs.cu", "latent_decode_umma.cu",
+    "selective_scan.cu",
 ]
 # the native reader of weight files (host code), loaded by the weights package
 IO_SOURCES = ["weight_reader.cu"]

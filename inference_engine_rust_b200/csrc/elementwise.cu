@@ -496,6 +496,32 @@ IERT_API int iert_gated_act_mul(const void* gu, void* out, int dtype, int n_toke
 }
 
 // ---------------------------------------------------------------------------------------
+// A projection's epilogue (IertEpilogue) on stored rows, in place: for products whose kernel does not take it.
+template <typename T>
+__global__ void epilogue_rows_kernel(T* __restrict__ z, long long ld, int cols, size_t total, IertEpilogue ep) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / cols;
+    const int n = (int)(i - t * cols);
+    T* o = z + t * ld + n;
+    *o = from_f32<T>(epilogue_value(to_f32(*o), (int)t, n, ep));
+  }
+}
+
+IERT_API int iert_epilogue_rows(void* z, int dtype, long long ld, int rows, int cols, const IertEpilogue* ep, cudaStream_t stream) {
+  if (rows <= 0 || cols <= 0) return IERT_OK;
+  if (!ep || (ep->scale && (ep->blocks < 0 || ep->block_cols <= 0))) return IERT_BAD_ARGUMENT;
+  const size_t total = (size_t)rows * cols, want = (total + 255) / 256, cap = (size_t)iert_sm_count_cached() * 16;
+  const dim3 blocks((unsigned)(want < cap ? want : cap));
+  if (dtype == IERT_F32) launch_dep(epilogue_rows_kernel<float>, blocks, dim3(256), 0, stream, (float*)z, ld, cols, total, *ep);
+  else if (dtype == IERT_BF16)
+    launch_dep(epilogue_rows_kernel<__nv_bfloat16>, blocks, dim3(256), 0, stream, (__nv_bfloat16*)z, ld, cols, total, *ep);
+  else return IERT_BAD_ARGUMENT;
+  return iert_check_launch("epilogue_rows");
+}
+
+// ---------------------------------------------------------------------------------------
 // residual[i] += y[i] in fp32 (src/ops/residual_add.rs:3-12).  Used by parts whose last
 // kernel cannot add into the residual stream itself.
 template <typename T>

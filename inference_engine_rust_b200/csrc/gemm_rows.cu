@@ -71,6 +71,7 @@ struct RowsParams {
   int* err;
   IertRowScale scale;                     // scale.sumsq != null: the outputs are multiplied by the rows' 1 / rms
   IertNormAhead ahead;                    // ahead.scaled_out != null (residual add): the next norm's first half
+  IertEpilogue ep;                        // mode 0: bias, activation and column scale of the outputs (see common.cuh)
   int trace_seq;
   int w_dynamic;                          // the matrix operand was written by the kernel in front: nothing is fetched before the wait
 };
@@ -260,6 +261,7 @@ gemm_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
         for (int w = 0; w < WARPS; ++w) v += red[((size_t)w * ROWS + row) * (NT * 8) + tok];
         if (p.scale.sumsq && tok < p.M) v *= rstd_s[tok];
         if (live) {
+          if (epilogue_on(p.ep)) v = epilogue_value(v, tok, n, p.ep);
           if (p.out_dtype == IERT_F32) {
             float* o = (float*)p.out + (long long)tok * p.ldo + n;
             if (p.mode == MODE_ADD_RESIDUAL) v += *o;
@@ -332,13 +334,15 @@ IERT_API int iert_gemm_rows_trace_read(unsigned long long* stamps, int* meta) {
 // IERT_BAD_ARGUMENT is returned and nothing is launched.  force_stages: 0 = choose.
 //   scale (optional)  the rows of x are the first half of an RMSNorm (IertNormAhead of the kernel that
 //                     wrote them): the outputs are multiplied by each row's 1 / rms (see common.cuh).
+//   ep (optional; mode 0)  bias, activation and column scale of the outputs (after `scale`).
 //   w_dynamic         w is no stored weight but rows that the kernel in front wrote (a few stored rows against many
 //                     tokens, the tokens as the streamed matrix): it is not fetched ahead of the dependency wait.
 //   ahead (optional; mode 1)  the first half of the NEXT norm over the new rows of `out`: ahead->parts
 //                     is set to the number of partial sums per row written (one per CTA).
 IERT_API int iert_gemm_rows(const void* x, long long ldx, const void* w, long long ldw, void* out, int out_dtype,
                             long long ldo, int M, int N, int K, int mode, const IertRowScale* scale,
-                            IertNormAhead* ahead, int force_stages, int w_dynamic, int* err, cudaStream_t stream) {
+                            IertNormAhead* ahead, const IertEpilogue* ep, int force_stages, int w_dynamic, int* err,
+                            cudaStream_t stream) {
   if (M <= 0 || N <= 0) return IERT_OK;
   if (M > 32 || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
     return IERT_BAD_ARGUMENT;
@@ -349,6 +353,7 @@ IERT_API int iert_gemm_rows(const void* x, long long ldx, const void* w, long lo
   if (ahead && (mode != MODE_ADD_RESIDUAL || !ahead->weight || !ahead->scaled_out || !ahead->sumsq_out ||
                 (ahead->weight_dtype != IERT_F32 && ahead->weight_dtype != IERT_BF16)))
     return IERT_BAD_ARGUMENT;
+  if (ep && (mode != MODE_STORE || (ep->scale && (ep->blocks < 0 || ep->block_cols <= 0)))) return IERT_BAD_ARGUMENT;
   const int nt = M <= 8 ? 1 : M <= 16 ? 2 : 4;
   RowsParams p;
   p.out = out; p.ldo = ldo; p.out_dtype = out_dtype; p.mode = mode;
@@ -356,6 +361,7 @@ IERT_API int iert_gemm_rows(const void* x, long long ldx, const void* w, long lo
   p.scale = IertRowScale{nullptr, 0, 0, 0.f};
   if (scale) p.scale = *scale;
   p.ahead = IertNormAhead{nullptr, 0, nullptr, 0, nullptr, 0};
+  p.ep = ep ? *ep : IertEpilogue{IERT_ACT_NONE, nullptr, nullptr, 0, 0, 1};
   p.kb_total = (K + KB - 1) / KB;
   p.n_stages = (p.kb_total + KPS - 1) / KPS;
   const int stage_bytes = KPS * (W_BYTES + nt * 8 * KB * 2);

@@ -83,6 +83,7 @@ struct GemmParams {
                         // the rows' 1 / rms
   IertNormAhead ahead;  // split-K residual add, tiles of 32 or 64 tokens: ahead.scaled_out != null: the reduction also
                         // writes the next norm's first half
+  IertEpilogue ep;      // plain stores: bias, activation and column scale of every output (see common.cuh)
   IertGatedAct act;     // gated launches: the activation (see common.cuh)
   int trace_seq;        // >= 0: the launch's row in the trace (builds with IERT_GEMM_TRACE only)
   uint32_t poll_limit;  // polls of a tile's counter before a CTA gives up waiting for the other CTAs of its tile
@@ -125,7 +126,8 @@ __device__ __forceinline__ void write_out_any(const GemmParams& p, int tok, int 
 }
 
 // Four consecutive outputs of one token, vectorised when aligned and inside the matrix.
-__device__ __forceinline__ void write_out4(const GemmParams& p, int tok, int n, const float4& r) {
+__device__ __forceinline__ void write_out4(const GemmParams& p, int tok, int n, float4 r) {
+  if (p.mode == MODE_STORE && epilogue_on(p.ep)) epilogue_run<4>(reinterpret_cast<float*>(&r), tok, n, p.N, p.ep);
   const bool whole = n + 4 <= p.N && (p.ldo & 3) == 0 && ((uintptr_t)p.out & 15) == 0;
   if (whole && p.out_dtype == IERT_F32) {
     float4* o = reinterpret_cast<float4*>((float*)p.out + (long long)tok * p.ldo + n);
@@ -511,6 +513,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
           float v[16];
           tmem_ld16(taddr + c, v);
           if (tok >= p.M) continue;
+          if (p.mode == MODE_STORE && epilogue_on(p.ep)) epilogue_run<16>(v, tok, n0 + c, p.N, p.ep);
           const bool full16 = n0 + c + 16 <= p.N;
           if (p.out_dtype == IERT_F32) {
             float* o = (float*)p.out + (long long)tok * p.ldo + n0 + c;
@@ -658,6 +661,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             for (int j = 0; j < 16; ++j)
               if (c + j < t_valid) o[(long long)j * p.ldo] = r[j] + v[j];
           } else {
+            if (epilogue_on(p.ep)) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                if (c + j < t_valid) v[j] = epilogue_value(v[j], t0 + c + j, n, p.ep);
+            }
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (c + j < t_valid) write_out_any(p, t0 + c + j, n, v[j]);
@@ -969,14 +977,15 @@ IERT_API int iert_gemm_tc_counter_count() { return 8192; }
 // x: [M, K] bf16, row stride ldx; w: [N, K] bf16, row stride ldw; out: [M, N] of out_dtype, row
 // stride ldo.  mode 0 stores, mode 1 adds into out.  K, ldx and ldw must be multiples of 8
 // and the pointers 16-byte aligned (TMA); otherwise IERT_BAD_ARGUMENT is returned and nothing
-// is launched.  ws / counters: scratch for split-K, shared by all launches on one stream;
+// is launched.  ep (optional, mode 0): bias, activation and column scale of the outputs.  ws / counters: scratch for split-K, shared by all launches on one stream;
 // counters must be zero before the first launch.  force_*: 0 = choose.
 namespace {
 int gemm_tc_impl(const void* x, long long ldx, const void* w, long long ldw, void* out, int out_dtype,
                  long long ldo, int M, int N, int K, int mode, float* ws, long long ws_bytes,
                  int* counters, int n_counters, int force_bt, int force_splits, int force_stages,
-                 const IertRowScale* scale, IertNormAhead* ahead, int* err, cudaStream_t stream) {
+                 const IertRowScale* scale, IertNormAhead* ahead, const IertEpilogue* ep, int* err, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return IERT_OK;
+  if (ep && (mode != MODE_STORE || scale || ahead || (ep->scale && (ep->blocks < 0 || ep->block_cols <= 0)))) return IERT_BAD_ARGUMENT;
   if (scale && (!scale->sumsq || scale->parts <= 0 || scale->hidden <= 0 || M > 64)) return IERT_BAD_ARGUMENT;
   if (ahead && (mode != MODE_ADD_RESIDUAL || M > 64 || !ahead->weight || !ahead->scaled_out || !ahead->sumsq_out ||
                 (ahead->weight_dtype != IERT_F32 && ahead->weight_dtype != IERT_BF16)))
@@ -1004,6 +1013,7 @@ int gemm_tc_impl(const void* x, long long ldx, const void* w, long long ldw, voi
   p.scale = IertRowScale{nullptr, 0, 0, 0.f};
   p.ahead = IertNormAhead{nullptr, 0, nullptr, 0, nullptr, 0};
   if (scale) p.scale = *scale;
+  p.ep = ep ? *ep : IertEpilogue{IERT_ACT_NONE, nullptr, nullptr, 0, 0, 1};
   p.tail_parts = 1; p.full_tiles = 0; p.tma_out = 0; p.t_group = 1 << 30;
   p.out = out; p.ldo = ldo; p.out_dtype = out_dtype; p.mode = mode;
   p.M = M; p.N = N; p.K = K;
@@ -1151,9 +1161,9 @@ IERT_API void iert_gemm_tc_set_poll_limit(unsigned int polls) { g_poll_limit = p
 IERT_API int iert_gemm_tc(const void* x, long long ldx, const void* w, long long ldw, void* out, int out_dtype,
                           long long ldo, int M, int N, int K, int mode, float* ws, long long ws_bytes,
                           int* counters, int n_counters, int force_bt, int force_splits, int force_stages,
-                          int* err, cudaStream_t stream) {
+                          const IertEpilogue* ep, int* err, cudaStream_t stream) {
   return gemm_tc_impl(x, ldx, w, ldw, out, out_dtype, ldo, M, N, K, mode, ws, ws_bytes, counters, n_counters, force_bt,
-                      force_splits, force_stages, nullptr, nullptr, err, stream);
+                      force_splits, force_stages, nullptr, nullptr, ep, err, stream);
 }
 
 // The same for one-token steps of 17 to 64 tokens whose input or output takes part in an RMSNorm split around
@@ -1168,7 +1178,7 @@ IERT_API int iert_gemm_tc_scaled(const void* x, long long ldx, const void* w, lo
                                  int* counters, int n_counters, const IertRowScale* scale, IertNormAhead* ahead,
                                  int force_bt, int force_splits, int* err, cudaStream_t stream) {
   return gemm_tc_impl(x, ldx, w, ldw, out, out_dtype, ldo, M, N, K, mode, ws, ws_bytes, counters, n_counters, force_bt,
-                      force_splits, 0, scale, ahead, err, stream);
+                      force_splits, 0, scale, ahead, nullptr, err, stream);
 }
 
 // act[t, i] = f(x[t] . w[i], x[t] . w[inter + i]) for w = [gate; up] of 2 * inter rows and f of the gated-activation
@@ -1184,6 +1194,7 @@ int gemm_tc_gated_impl(const void* x, long long ldx, const void* w, long long ld
   if (scale && (!scale->sumsq || scale->parts <= 0 || scale->hidden <= 0)) return IERT_BAD_ARGUMENT;
   GemmParams p;
   p.scale = IertRowScale{nullptr, 0, 0, 0.f};
+  p.ep = IertEpilogue{IERT_ACT_NONE, nullptr, nullptr, 0, 0, 1};
   p.tail_parts = 1; p.full_tiles = 0; p.tma_out = 0; p.t_group = 1 << 30;
   p.out = act; p.ldo = ldo; p.out_dtype = IERT_BF16; p.mode = MODE_GATED_SILU;
   p.act = fn ? *fn : IertGatedAct{INFINITY, INFINITY, 0.f, 1.f, 0.f};

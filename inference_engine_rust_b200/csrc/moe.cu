@@ -63,26 +63,40 @@ __global__ void router_topk_kernel(const float* __restrict__ z, long long ldz, c
     }
 }
 
-// one warp per token; shared memory: s[N], c[N], group score [groups], flags [N] (bytes).  Output e of token t is
+// A block per token, whose first warp routes; shared memory: s[N], c[N], group score [groups], flags [N] (bytes).  Output e of token t is
 // z[t * ldz + e * lde]: rows of tokens (lde = 1) or rows of outputs (ldz = 1).
 //   score_mode   0: scores are the softmax over all N outputs; 1: every output's own sigmoid
 //   group_mode   0: a group's score is its best choice score; 1: the sum of its two best (of its one, if it has one)
-//   weights      chosen scores / (their sum + weight_eps) * weight_scale
-__global__ void router_grouped_kernel(const float* __restrict__ z, long long ldz, long long lde, const float* __restrict__ correction, int E,
-                                      int N, int top, int groups, int keep, int score_mode, int group_mode, float weight_eps,
-                                      float weight_scale, float* __restrict__ wt, float* __restrict__ wid,
-                                      int* __restrict__ idx, float* __restrict__ w) {
-  extern __shared__ float rsm[];
+//   weights      chosen scores / (their sum + weight_eps) * weight_scale; with renorm 0 chosen scores * weight_scale
+//   ldw          row stride of wt; with shared_gate the output behind the last (number N) is the logit of a gate on an expert
+//                every token uses: wt[t, E] = sigmoid(z[N]) (ldw > E)
+//   x, residual  (optional) the identity experts' share is added here: residual[t] += wid[t] * x[t], by all the block's warps
+struct RouterArgs {
+  const float* z;
+  long long ldz, lde;
+  const float* correction;
+  int E, N, top, groups, keep, score_mode, group_mode;
+  float weight_eps, weight_scale;
+  int renorm, shared_gate, ldw;
+  float* wt;
+  float* wid;
+  int* idx;
+  float* w;
+};
+
+// The routing of token t by one warp; returns the identity experts' share (in lane 0).
+__device__ __forceinline__ float route_token(const RouterArgs& a, int t, int lane, float* rsm) {
+  const int E = a.E, N = a.N, top = a.top, groups = a.groups, keep = a.keep;
+  const long long lde = a.lde;
   float* s = rsm;
   float* c = rsm + N;
   float* gs = rsm + 2 * N;
   unsigned char* open = reinterpret_cast<unsigned char*>(rsm + 2 * N + groups);      // 1: may still be chosen
-  pdl_launch_dependents();     // the next kernel (the experts' product) may fetch its first weights now
-  pdl_wait();
-  const int t = blockIdx.x, lane = threadIdx.x, per = N / groups;
-  const float* row = z + (size_t)t * ldz;
+  const int per = N / groups;
+  const float* row = a.z + (size_t)t * a.ldz;
+  const float* correction = a.correction;
   float den = 1.f;
-  if (score_mode == 0) {
+  if (a.score_mode == 0) {
     float m = -INFINITY;
     for (int e = lane; e < N; e += 32) m = fmaxf(m, row[e * lde]);
     m = warp_max(m);
@@ -105,7 +119,7 @@ __global__ void router_grouped_kernel(const float* __restrict__ z, long long ldz
       if (v > best) { second = best; best = v; }
       else if (v > second) second = v;
     }
-    gs[g] = group_mode == 1 && per > 1 ? best + second : best;
+    gs[g] = a.group_mode == 1 && per > 1 ? best + second : best;
   }
   __syncwarp();
   // the `keep` best groups, one after the other; a group that was taken is marked by NaN
@@ -152,19 +166,60 @@ __global__ void router_grouped_kernel(const float* __restrict__ z, long long ldz
     if (lane == 0 && bi != 0x7fffffff) open[bi] = 0;
     __syncwarp();
   }
-  for (int e = lane; e < E; e += 32) wt[(size_t)t * E + e] = 0.f;
+  float* wt = a.wt + (size_t)t * a.ldw;
+  for (int e = lane; e < E; e += 32) wt[e] = 0.f;
   __syncwarp();
+  float identity = 0.f;
   if (lane == 0) {
-    float identity = 0.f;
     for (int k = 0; k < top; ++k) {
-      const float p = val[k] / (sum + weight_eps) * weight_scale;
-      if (chosen[k] < E) wt[(size_t)t * E + chosen[k]] = p;
+      const float p = a.renorm ? val[k] / (sum + a.weight_eps) * a.weight_scale : val[k] * a.weight_scale;
+      if (chosen[k] < E) wt[chosen[k]] = p;
       else if (chosen[k] < N) identity += p;
-      idx[(size_t)t * top + k] = chosen[k] < N ? chosen[k] : -1;
-      w[(size_t)t * top + k] = p;
+      a.idx[(size_t)t * top + k] = chosen[k] < N ? chosen[k] : -1;
+      a.w[(size_t)t * top + k] = p;
     }
-    wid[t] = identity;
+    a.wid[t] = identity;
+    if (a.shared_gate) wt[E] = 1.0f / (1.0f + expf(-row[N * lde]));
   }
+  return identity;
+}
+
+template <typename TX>
+__global__ void router_grouped_kernel(RouterArgs a, const TX* __restrict__ x, long long ldx, float* __restrict__ residual, int H) {
+  extern __shared__ float rsm[];
+  __shared__ float share_s;
+  pdl_launch_dependents();     // the next kernel (the experts' product) may fetch its first weights now
+  pdl_wait();
+  const int t = blockIdx.x;
+  if (threadIdx.x < 32) {
+    const float share = route_token(a, t, threadIdx.x, rsm);
+    if (threadIdx.x == 0) share_s = share;
+  }
+  if (!x) return;
+  __syncthreads();
+  const float share = share_s;
+  if (share == 0.f) return;
+  float* out = residual + (size_t)t * H;
+  const TX* in = x + (size_t)t * ldx;
+  if (H % 4 == 0 && ldx % 4 == 0 && (((uintptr_t)residual | (uintptr_t)x) & 15) == 0) {
+    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+      float4 o = *reinterpret_cast<const float4*>(out + i);
+      float v[4];
+      if (sizeof(TX) == 2) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(in + i);
+        const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        v[0] = f0.x; v[1] = f0.y; v[2] = f1.x; v[3] = f1.y;
+      } else {
+        const float4 f = *reinterpret_cast<const float4*>(in + i);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+      }
+      o.x += share * v[0]; o.y += share * v[1]; o.z += share * v[2]; o.w += share * v[3];
+      *reinterpret_cast<float4*>(out + i) = o;
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] += share * to_f32(in[i]);
 }
 
 template <typename T>
@@ -208,19 +263,27 @@ IERT_API int iert_router_topk(const float* z, long long ldz, const float* bias, 
   return iert_check_launch("router_topk");
 }
 
-// z: output e of token t at z[t * ldz + e * lde] (fp32).
+// z: output e of token t at z[t * ldz + e * lde] (fp32).  x (optional, [n_tokens, H] of x_dtype) with residual (fp32 [n_tokens, H]): the
+// identity experts' share is added there.
 IERT_API int iert_router_grouped(const float* z, long long ldz, long long lde, const float* correction, int n_tokens, int E, int N, int top,
                                  int groups, int keep, int score_mode, int group_mode, float weight_eps, float weight_scale,
-                                 float* wt, float* wid, int* idx, float* w, cudaStream_t stream) {
+                                 int renorm, int shared_gate, float* wt, int ldw, float* wid, int* idx, float* w, const void* x,
+                                 int x_dtype, long long ldx, float* residual, int H, cudaStream_t stream) {
   if (n_tokens <= 0) return IERT_OK;
   if (score_mode < 0 || score_mode > 1 || group_mode < 0 || group_mode > 1) return IERT_BAD_ARGUMENT;
+  if (ldw < E + (shared_gate ? 1 : 0) || (x && (!residual || H <= 0 || (x_dtype != IERT_F32 && x_dtype != IERT_BF16)))) return IERT_BAD_ARGUMENT;
   if (E < 0 || N < E || N <= 0 || top <= 0 || top > MAX_TOP || groups <= 0 || N % groups || keep <= 0 || keep > groups ||
       top > keep * (N / groups))
     return IERT_BAD_ARGUMENT;
   const size_t smem = (size_t)(2 * N + groups) * sizeof(float) + (size_t)N;
   if (smem > 48 * 1024) return IERT_BAD_ARGUMENT;
-  launch_dep(router_grouped_kernel, dim3(n_tokens), dim3(32), smem, stream, z, ldz, lde, correction, E, N, top, groups, keep, score_mode,
-             group_mode, weight_eps, weight_scale, wt, wid, idx, w);
+  const RouterArgs a = {z, ldz, lde, correction, E, N, top, groups, keep, score_mode, group_mode, weight_eps, weight_scale, renorm,
+                        shared_gate, ldw, wt, wid, idx, w};
+  const dim3 threads(x ? 256 : 32);
+  if (x && x_dtype == IERT_F32)
+    launch_dep(router_grouped_kernel<float>, dim3(n_tokens), threads, smem, stream, a, (const float*)x, ldx, residual, H);
+  else
+    launch_dep(router_grouped_kernel<__nv_bfloat16>, dim3(n_tokens), threads, smem, stream, a, (const __nv_bfloat16*)x, ldx, residual, H);
   return iert_check_launch("router_grouped");
 }
 

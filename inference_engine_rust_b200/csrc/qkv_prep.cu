@@ -9,6 +9,8 @@
 //   bias     (optional) fp32 [heads*dim + kv_heads*dim + kv_heads*vdim], added to the projection
 //   wq, wk   (optional) fp32 [dim]: every head of q (of k) is divided by its root mean square, eps inside the
 //            root, and multiplied by this weight, the same for all heads; before the rotation
+//   temperature (optional, temp_every > 0): every head of q is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1), p the
+//            token's position
 //   rotation of the first `rotary_dim` numbers of every head of q and k by position * inv_freq[i], cosine and sine
 //            multiplied by rot_mul; pairing
 //            "half": number i with number i + rotary_dim / 2; "interleaved": number 2i with number 2i + 1
@@ -26,12 +28,16 @@ namespace {
 constexpr int WARPS = 8;
 constexpr int THREADS = WARPS * 32;
 
+__device__ __forceinline__ float query_temperature(int pos, float coef, float every) {
+  return 1.0f + coef * logf(floorf(((float)pos + 1.0f) / every) + 1.0f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(THREADS)
 qkv_prep_kernel(const float* __restrict__ proj, long long ld, const float* __restrict__ bias, T* __restrict__ qkv,
                 IertBatchView b, IertKvView c, int heads, int dim, int vdim, const float* __restrict__ inv_freq,
                 int rotary_dim, float rot_mul, int pairing, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
-                const float* __restrict__ v0, long long ldv0, float lam, int write_cache, int* __restrict__ err) {
+                const float* __restrict__ v0, long long ldv0, float lam, float temp_coef, float temp_every, int write_cache, int* __restrict__ err) {
   extern __shared__ float sm[];
   pdl_launch_dependents();
   const int D = c.head_dim, nkv = c.kv_heads, half = rotary_dim / 2;
@@ -53,6 +59,7 @@ qkv_prep_kernel(const float* __restrict__ proj, long long ld, const float* __res
   const int q_begin = b.cu_q[s], q_len = b.cu_q[s + 1] - q_begin;
   const int pos = b.pos0[s] + (t - q_begin);
   const int final_len = b.pos0[s] + q_len;
+  const float q_mul = temp_every > 0.f ? query_temperature(pos, temp_coef, temp_every) : 1.0f;
   for (int k = threadIdx.x; k < half; k += THREADS) {
     float sn, co;
     sincosf((float)pos * inv_freq[k], &sn, &co);
@@ -83,6 +90,8 @@ qkv_prep_kernel(const float* __restrict__ proj, long long ld, const float* __res
       const float r = 1.0f / sqrtf(ss / (float)dim + eps);
       for (int d = lane; d < n; d += 32) v[d] = v[d] * r * w[d];
     }
+    if (temp_every > 0.f && h < heads)
+      for (int d = lane; d < n; d += 32) v[d] *= q_mul;
     __syncwarp();
     if (!is_v) {
       for (int k = lane; k < half; k += 32) {
@@ -125,7 +134,7 @@ __global__ void __launch_bounds__(THREADS)
 qkv_prep_vec_kernel(const float* __restrict__ proj, long long ld, const float* __restrict__ bias, T* __restrict__ qkv,
                     IertBatchView b, IertKvView c, int heads, int dim, int vdim, const float* __restrict__ inv_freq,
                     int rotary_dim, float rot_mul, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
-                    const float* __restrict__ v0, long long ldv0, float lam, int write_cache, int* __restrict__ err) {
+                    const float* __restrict__ v0, long long ldv0, float lam, float temp_coef, float temp_every, int write_cache, int* __restrict__ err) {
   extern __shared__ float sm[];
   pdl_launch_dependents();
   const int D = c.head_dim, nkv = c.kv_heads, half = rotary_dim / 2;
@@ -144,6 +153,7 @@ qkv_prep_vec_kernel(const float* __restrict__ proj, long long ld, const float* _
   const int q_begin = b.cu_q[s], q_len = b.cu_q[s + 1] - q_begin;
   const int pos = b.pos0[s] + (t - q_begin);
   const int final_len = b.pos0[s] + q_len;
+  const float q_mul = temp_every > 0.f ? query_temperature(pos, temp_coef, temp_every) : 1.0f;
   for (int k = threadIdx.x; k < half; k += THREADS) {
     float sn, co;
     sincosf((float)pos * inv_freq[k], &sn, &co);
@@ -193,6 +203,10 @@ qkv_prep_vec_kernel(const float* __restrict__ proj, long long ld, const float* _
           x[j].x = x[j].x * r * ww.x; x[j].y = x[j].y * r * ww.y; x[j].z = x[j].z * r * ww.z; x[j].w = x[j].w * r * ww.w;
         }
       }
+    }
+    if (temp_every > 0.f && h < heads) {
+#pragma unroll
+      for (int j = 0; j < CH; ++j) { x[j].x *= q_mul; x[j].y *= q_mul; x[j].z *= q_mul; x[j].w *= q_mul; }
     }
     if (HALF && !is_v) {
       float* row = cs + rotary_dim + warp * rotary_dim;     // 16-byte aligned: rotary_dim is a multiple of 8
@@ -306,7 +320,7 @@ __global__ void gate_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ attn, c
 IERT_API int iert_qkv_prep(const float* proj, long long ld, const float* bias, void* qkv, int dtype, const IertBatchView* batch,
                            const IertKvView* cache, int heads, int dim, int vdim, const float* inv_freq, int rotary_dim,
                            float rot_mul, int pairing, const float* wq, const float* wk, float eps, const float* v0, long long ldv0,
-                           float lam, int write_cache, int* err, cudaStream_t stream) {
+                           float lam, float temp_coef, float temp_every, int write_cache, int* err, cudaStream_t stream) {
   if (batch->n_tokens <= 0) return IERT_OK;
   const int D = cache->head_dim;
   if (dim <= 0 || vdim <= 0 || dim > D || vdim > D || rotary_dim < 0 || rotary_dim > dim || (rotary_dim & 1) ||
@@ -331,10 +345,10 @@ IERT_API int iert_qkv_prep(const float* proj, long long ld, const float* bias, v
     do {                                                                                                               \
       if (half_pairs)                                                                                                  \
         launch_dep(qkv_prep_vec_kernel<T, CH, true>, grid, dim3(THREADS), vsmem, stream, proj, ld, bias, (T*)qkv, *batch, *cache, \
-                   heads, dim, vdim, inv_freq, rotary_dim, rot_mul, wq, wk, eps, v0, ldv0, lam, write_cache, err);     \
+                   heads, dim, vdim, inv_freq, rotary_dim, rot_mul, wq, wk, eps, v0, ldv0, lam, temp_coef, temp_every, write_cache, err);     \
       else                                                                                                             \
         launch_dep(qkv_prep_vec_kernel<T, CH, false>, grid, dim3(THREADS), vsmem, stream, proj, ld, bias, (T*)qkv, *batch, *cache, \
-                   heads, dim, vdim, inv_freq, rotary_dim, rot_mul, wq, wk, eps, v0, ldv0, lam, write_cache, err);     \
+                   heads, dim, vdim, inv_freq, rotary_dim, rot_mul, wq, wk, eps, v0, ldv0, lam, temp_coef, temp_every, write_cache, err);     \
     } while (0)
     if (dtype == IERT_F32) { if (D <= 128) GO(float, 1); else GO(float, 2); }
     else { if (D <= 128) GO(__nv_bfloat16, 1); else GO(__nv_bfloat16, 2); }
@@ -343,10 +357,10 @@ IERT_API int iert_qkv_prep(const float* proj, long long ld, const float* bias, v
   }
   if (dtype == IERT_F32)
     launch_dep(qkv_prep_kernel<float>, grid, dim3(THREADS), smem, stream, proj, ld, bias, (float*)qkv, *batch, *cache, heads, dim,
-               vdim, inv_freq, rotary_dim, rot_mul, pairing, wq, wk, eps, v0, ldv0, lam, write_cache, err);
+               vdim, inv_freq, rotary_dim, rot_mul, pairing, wq, wk, eps, v0, ldv0, lam, temp_coef, temp_every, write_cache, err);
   else if (dtype == IERT_BF16)
     launch_dep(qkv_prep_kernel<__nv_bfloat16>, grid, dim3(THREADS), smem, stream, proj, ld, bias, (__nv_bfloat16*)qkv, *batch,
-               *cache, heads, dim, vdim, inv_freq, rotary_dim, rot_mul, pairing, wq, wk, eps, v0, ldv0, lam, write_cache, err);
+               *cache, heads, dim, vdim, inv_freq, rotary_dim, rot_mul, pairing, wq, wk, eps, v0, ldv0, lam, temp_coef, temp_every, write_cache, err);
   else
     return IERT_BAD_ARGUMENT;
   return iert_check_launch("qkv_prep");

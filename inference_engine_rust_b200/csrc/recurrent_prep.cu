@@ -106,7 +106,8 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(DeltaPrepArgs a, IertBa
     for (int h = lane; h < a.H; h += 32) {
       const float gb = a.gates[(size_t)t * a.gld + h], ga = a.gates[(size_t)t * a.gld + a.H + h];
       a.beta[(size_t)t * a.H + h] = sigmoid_f(gb);
-      a.decay[(size_t)t * a.H + h] = expf(-expf(a.A_log[h]) * softplus_f(ga + a.dt_bias[h]));
+      // 1 + expm1: a decay near 1 keeps its distance from 1, whose error a long sequence would gather
+      a.decay[(size_t)t * a.H + h] = 1.0f + expm1f(-expf(a.A_log[h]) * softplus_f(ga + a.dt_bias[h]));
     }
 }
 

@@ -45,6 +45,10 @@ class Model:
         self.embedding: Optional[torch.Tensor] = None
         self.lm_head = part_class("head", spec.head.kind)(spec.head, h, spec.vocab_size, rt)
         self.inputs = [(part_class("input", ps.kind)(ps, h, spec.vocab_size, rt), prefix) for ps, prefix in spec.inputs]
+        self.passes, self._passes_prefix = None, ""
+        if spec.passes is not None:
+            ps, self._passes_prefix = spec.passes
+            self.passes = part_class("pass", ps.kind)(ps, h, rt)
         self.loaded = False
         # called after every scheduled layer with (its position, the residual rows or streams, the step's
         # context): for looking at the residual between layers; runs inside the step, so it must launch on
@@ -82,6 +86,9 @@ class Model:
         for part, prefix in self.inputs:
             for local, ts in part.tensor_specs().items():
                 out[prefix + local] = ts
+        if self.passes is not None:
+            for local, ts in self.passes.tensor_specs().items():
+                out[self._passes_prefix + local] = ts
         for ls, (norm1, mixer, norm2, ffn), extra, block in zip(spec.layers, self._layer_parts, self._extra_norms,
                                                                 self.blocks):
             out.update(self._norm_specs(norm1, ls.mixer_norm_name))
@@ -140,6 +147,8 @@ class Model:
             self.embedding = tied                          # tied: one copy
         for part, prefix in self.inputs:
             part.load({local: get(prefix + local) for local in part.tensor_specs()})
+        if self.passes is not None:
+            self.passes.load({local: get(self._passes_prefix + local) for local in self.passes.tensor_specs()})
         for ls, (norm1, mixer, norm2, ffn), extra, block in zip(spec.layers, self._layer_parts, self._extra_norms,
                                                                 self.blocks):
             load_norm(norm1, ls.mixer_norm_name)
@@ -184,6 +193,8 @@ class Model:
         """True when every part declares `graph_safe`: its forward reads the step's sequences
         from device memory only, so a captured launch sequence stays right for later steps."""
         parts = [self.final_norm, self.lm_head] + [part for part, _ in self.inputs]
+        if self.passes is not None:
+            parts.append(self.passes)
         for e in self.spec.schedule:
             parts.extend(p for p in self._layer_parts[e.layer] if p is not None)
             parts.extend(self._extra_norms[e.layer].values())
@@ -193,7 +204,8 @@ class Model:
     def weight_bytes_per_step(self) -> int:
         """Bytes of weights a one-token step reads: every matrix each scheduled layer uses,
         the norm scales, the output head (the embedding rows it gathers are negligible)."""
-        total = self.lm_head.nbytes() + sum(part.weight_bytes() for part, _ in self.inputs if hasattr(part, "weight_bytes"))
+        others = [part for part, _ in self.inputs] + [self.passes]
+        total = self.lm_head.nbytes() + sum(part.weight_bytes() for part in others if hasattr(part, "weight_bytes"))
         for e in self.spec.schedule:
             norm1, mixer, norm2, ffn = self._layer_parts[e.layer]
             for part in (mixer, ffn):
@@ -235,8 +247,9 @@ class Model:
         x = ws.take("model.residual", (T, H), torch.float32)
         sched = spec.schedule
         # the first block's first norm may ask the embedding kernel for its element-wise half
-        # (not when step inputs may still change the embedded rows)
-        request = first_norm_request_of(self.blocks[sched[0].layer], ctx) if sched and not self.inputs else None
+        # (not when step inputs or the start of a pass may still change the embedded rows)
+        begins = bool(sched) and sched[0].pass_start is not None
+        request = first_norm_request_of(self.blocks[sched[0].layer], ctx) if sched and not self.inputs and not begins else None
         ahead = finish = None
         if request is not None:
             from ..parts.norm import honour
@@ -252,6 +265,8 @@ class Model:
             else:
                 part.prepare(tokens, x, ctx)
         ctx.input_view = None
+        if self.passes is not None:
+            self.passes.embedded(x, ctx, begins)
         S = spec.residual_streams
         rows = x
         if S is not None:
@@ -260,7 +275,11 @@ class Model:
             B.streams_expand(x, rows, T, S, H, ctx.stream)
         for pos, e in enumerate(sched):
             view = cache.layer_view(spec.cache_entry(pos))
-            ctx.next_block = self.blocks[sched[pos + 1].layer] if pos + 1 < len(sched) else None
+            if e.pass_start is not None:
+                self.passes.begin(e.pass_start, rows, ctx, self.blocks[e.layer], pos == 0)
+            # no block prepares rows for a layer in front of which the start of a pass changes them
+            last = pos + 1 == len(sched) or sched[pos + 1].pass_start is not None
+            ctx.next_block = None if last else self.blocks[sched[pos + 1].layer]
             self.blocks[e.layer].forward(rows, ctx, view, e.writes_cache)
             if self.after_block is not None:
                 self.after_block(pos, rows, ctx)

@@ -12,6 +12,7 @@ kind; the configuration then names that kind for the layers that use it.
     block     Block(layer_spec, norm1, mixer, norm2, ffn, rt[, extra_norms={role: norm}])   .forward(x, ctx, cache_view, writes_cache)
     head      Head(spec, hidden_size, vocab_size, rt)   .forward(hn, logits_f32, n_rows, ctx)
     input     StepInput(spec, hidden_size, vocab_size, rt)   .prepare(tokens, x_f32, ctx)
+    pass      PassStart(spec, hidden_size, rt)   .embedded(x_f32, ctx, begins_here)   .begin(t, x_f32, ctx, block, first)
 
 Optional, for one-token steps (see `NormRequest`, `LazyInput`): a norm may let the kernel that writes
 its input rows do its element-wise half and the projection that reads its output its row-wise half.
@@ -31,7 +32,7 @@ from ..config.specs import LayerSpec, PartSpec
 from ..weights.loader import TensorSpec
 
 _REGISTRY: Dict[Tuple[str, str], type] = {}
-CATEGORIES = ("norm", "position", "mixer", "ffn", "block", "head", "input")
+CATEGORIES = ("norm", "position", "mixer", "ffn", "block", "head", "input", "pass")
 
 
 def register_part(category: str, kind: str, cls: type, *, replace: bool = False) -> None:
@@ -285,6 +286,21 @@ class Head(Part):
 
     def nbytes(self) -> int:
         """Bytes of weights a step reads through this head."""
+        raise NotImplementedError
+
+
+class PassStart(Part):
+    """Changes the residual rows right before the first layer of each pass of a run of layers that is executed several
+    times (the schedule entries with a `pass_start`).  Its tensors are found under the prefix that `ModelSpec.passes` names
+    beside its spec."""
+
+    def embedded(self, x, ctx: StepContext, begins_here: bool) -> None:
+        """Called once per step with the embedded rows (after the step inputs); `begins_here`: the first scheduled entry
+        starts a pass, so `begin` is called on these rows next."""
+
+    def begin(self, t: int, x, ctx: StepContext, block, first: bool) -> None:
+        """Pass number `t` starts: change `x` in place (`first`: these are still the embedded rows).  `block` runs next; if
+        it has `begin_rows(x, ctx, e=, step=, keep=)`, it can do the addition together with its own first norm."""
         raise NotImplementedError
 
 

@@ -1,6 +1,7 @@
 """Arrangement of a layer's parts.  "two_norms": x += mixer(norm1(x)) + ffn(norm2(x)), both norms of the same
 x.  "shared_norm": h = norm1(x); x += mixer(h) + ffn(h) (one norm, read by both
-sublayers).  "prenorm": x += mixer(norm1(x)); x += ffn(norm2(x)) (the second
+sublayers).  "sandwich": a norm on both sides of each
+sublayer.  "prenorm": x += mixer(norm1(x)); x += ffn(norm2(x)) (the second
 half left out for a layer without a feed-forward)
 (src/layers/block.rs:19-24,63-65; the residual uses the un-normed input,
 src/layers/attention.rs:757-759, src/layers/ffn.rs:113-116)."""
@@ -168,6 +169,56 @@ class OutputNormBlock(Block):
         ctx.rows_ahead = CastAhead(x, h, y)
 
 
+class SandwichBlock(Block):
+    """A norm on both sides of each sublayer, m being the block's `factor`:
+
+        x <- x + m post1(mixer(norm1(x)));   x <- x + m post2(ffn(norm2(x)))      (the second half left out without a feed-forward)
+
+    post1 and post2 are the layer's extra norms "mixer_out" and "ffn_out".  The sublayers add into a zeroed fp32 buffer y;
+    one kernel per sublayer norms y, adds it to the fp32 residual, clears y and norms the new residual for the sublayer to
+    come, also across the block boundary (the next block of this kind finds its input ready)."""
+    graph_safe = True
+
+    def __init__(self, layer_spec, norm1, mixer, norm2, ffn, rt: Runtime, extra_norms):
+        self.norm1, self.mixer, self.norm2, self.ffn, self.rt = norm1, mixer, norm2, ffn, rt
+        self.post1, self.post2 = extra_norms["mixer_out"], extra_norms.get("ffn_out")
+        self.factor = float(layer_spec.block.get("factor", 1.0))
+        if ffn is not None and (norm2 is None or self.post2 is None):
+            raise ValueError("block 'sandwich' with a feed-forward needs a second norm and an extra norm 'ffn_out'")
+        for n in (norm1, norm2, self.post1, self.post2):
+            if n is not None and not hasattr(n, "begin_rows"):
+                raise ValueError(f"block 'sandwich' needs norms with add_normed and begin_rows, got {type(n).__name__}")
+
+    def _buffers(self, x):
+        ws = self.rt.workspace
+        return ws.take("block.normed", x.shape, self.rt.dtype), ws.take("block.sublayer_out", x.shape, torch.float32)
+
+    def begin_rows(self, x, ctx: StepContext, e=None, step=None, keep=None) -> None:
+        """x <- x + e + step in the kernel that does this block's first norm (`keep` receives the rows as they were)."""
+        h, y = self._buffers(x)
+        self.norm1.begin_rows(x, h, ctx, ctx.n_tokens, clear=y, e=e, step=step, keep=keep)
+        ctx.rows_ahead = NormedAhead(self.norm1, x, h)
+
+    def forward(self, x, ctx: StepContext, cache_view, writes_cache: bool) -> None:
+        T = ctx.n_tokens
+        ctx.norm_ahead = None
+        h, y = self._buffers(x)
+        ahead, ctx.rows_ahead = ctx.rows_ahead, None
+        if not (isinstance(ahead, NormedAhead) and ahead.norm is self.norm1 and ahead.rows is x
+                and ahead.normed.data_ptr() == h.data_ptr() and ahead.normed.dtype == h.dtype):
+            self.norm1.begin_rows(x, h, ctx, T, clear=y)
+        nxt = ctx.next_block
+        after = nxt.norm1 if isinstance(nxt, SandwichBlock) else None
+        self.mixer.forward(h, y, ctx, cache_view, writes_cache)
+        if self.ffn is not None:
+            self.post1.add_normed(y, x, h, ctx, T, self.factor, then=self.norm2)
+            self.ffn.forward(h, y, ctx)
+        last = self.post1 if self.ffn is None else self.post2
+        last.add_normed(y, x, h if after is not None else None, ctx, T, self.factor, then=after)
+        if after is not None:
+            ctx.rows_ahead = NormedAhead(after, x, h)
+
+
 class SharedNormBlock(Block):
     """One norm, read by both sublayers, whose results are added to the same residual:
 
@@ -239,4 +290,5 @@ register_part("block", "prenorm", PreNormBlock)
 register_part("block", "two_norms", TwoNormsBlock)
 register_part("block", "shared_norm", SharedNormBlock)
 register_part("block", "outnorm", OutputNormBlock)
+register_part("block", "sandwich", SandwichBlock)
 register_part("block", "hyper", HyperConnectionBlock)

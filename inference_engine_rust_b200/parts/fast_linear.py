@@ -35,15 +35,18 @@ def norm_ahead_enabled() -> bool:
 NORM_AHEAD_MAX_TOKENS = 64
 
 
-def apply(linear, x, out, n_rows: int, mode: int, stream: int, ctx=None) -> bool:
+def apply(linear, x, out, n_rows: int, mode: int, stream: int, ctx=None, epilogue=None) -> bool:
     """Run the tensor-core product if it takes these operands (bf16, K and row strides
     multiples of 8, 16-byte aligned); False means nothing was launched and the caller runs the
     plain kernel.  `x` may be the first half of a norm (`ScaledRows`); `ctx` (residual adds): its
-    `norm_ahead`, if set, is honoured where the kernel can and the result left in `ctx.rows_ahead`."""
+    `norm_ahead`, if set, is honoured where the kernel can and the result left in `ctx.rows_ahead`.  `epilogue` (plain
+    stores): what the kernel does to the outputs."""
     from .norm import ScaledRows, honour
     if linear.weight.dtype != torch.bfloat16:
         return False
     err = linear.rt.err
+    if epilogue is not None:
+        x = as_tensor(x, n_rows)
     scaled = x if isinstance(x, ScaledRows) else None
     request = ctx.norm_ahead if ctx is not None and mode == B.GEMM_ADD_RESIDUAL else None
     thin = 2 * -(-linear.out_features // 128) <= 2 * B.sm_count()       # 128-row tiles alone would not fill the device
@@ -56,7 +59,7 @@ def apply(linear, x, out, n_rows: int, mode: int, stream: int, ctx=None) -> bool
                 ahead, finish = honour(request, out, ctx, "linear", parts)
             scale = scaled.row_scale() if scaled is not None else None
             if n_rows <= ROWS_KERNEL_MAX_TOKENS:
-                done = B.gemm_rows(xt, linear.weight, out, n_rows, mode, err, stream, scale=scale, ahead=ahead)
+                done = B.gemm_rows(xt, linear.weight, out, n_rows, mode, err, stream, scale=scale, ahead=ahead, epilogue=epilogue)
             else:
                 done = (scale is not None or ahead is not None) and \
                     B.gemm_tc_scaled(xt, linear.weight, out, n_rows, mode, err, stream, scale=scale, ahead=ahead)
@@ -67,7 +70,9 @@ def apply(linear, x, out, n_rows: int, mode: int, stream: int, ctx=None) -> bool
     x = as_tensor(x, n_rows)
     if x.dtype != torch.bfloat16:
         return False
-    return B.gemm_tc(x, linear.weight, out, n_rows, mode, err, stream)
+    # (a forced token tile keeps a prompt's plain store off the token-major kernel, which does not split the inner axis)
+    return B.gemm_tc(x, linear.weight, out, n_rows, mode, err, stream, force_bt=256 if linear.narrow and n_rows > 256 else 0,
+                     epilogue=epilogue)
 
 
 def apply_gated(linear, x, act, n_rows: int, stream: int, fn=None) -> bool:

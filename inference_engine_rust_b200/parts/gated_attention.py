@@ -11,13 +11,16 @@ concatenated heads or on each head:
     v <- (1 - lambda) v + lambda v_first                                      (`v_mix` "mix": v_first are the values, as
                                                                                projected, of the layer with `v_mix` "source",
                                                                                for the same token; the mixed v is cached)
+    q <- q (1 + coef ln(floor((p + 1) / every) + 1))                          (`q_temp` {coef, every}: p is the position)
     a = softmax(q . k * scale over the visible keys) v                        (causal, optionally a sliding `window` behind
-                                                                               which the first `keep` positions stay visible)
+                                                                               which the first `keep` positions stay visible;
+                                                                               `sink`: exp(sink_h) in the denominator, with
+                                                                               no key and no value, not scaled)
     y = W_o (a * sigmoid(W_g h))                                              (`gate` True: a gate per number; "head": one
                                                                                per head, the same for all its numbers)
 
 Tensors: q, k, v (+ q.b, k.b, v.b), q.norm, k.norm, vmix (one number; the source layer has it too and does not use it),
-g, o.  One product makes [q | k | v | g] in fp32; one kernel adds
+sink [heads], g, o.  One product makes [q | k | v | g] in fp32; one kernel adds
 the biases, norms, rotates, rounds once and writes the packed row and the cache; the library's attention kernels run
 on heads padded with zeros to one common size D >= max(head_dim, v_dim) (a multiple of 16 for the tensor-core kernels),
 so that keys and values share the paged cache's geometry; one kernel drops the padding and applies the gate; W_o adds
@@ -59,6 +62,9 @@ class GatedAttention(Mixer):
         if self.v_mix not in (None, "source", "mix"):
             raise ValueError(f"v_mix must be 'source', 'mix' or None, got {self.v_mix!r}")
         self.lam = 0.0
+        self.has_sink, self.sink = bool(spec.get("sink", False)), None
+        temp = spec.get("q_temp")
+        self.temp_coef, self.temp_every = (0.0, 0.0) if temp is None else (float(temp["coef"]), float(temp["every"]))
         qk_norm = spec.get("qk_norm")
         if qk_norm not in (None, "head"):
             raise ValueError(f"qk_norm must be 'head' or None, got {qk_norm!r}")
@@ -91,6 +97,8 @@ class GatedAttention(Mixer):
             specs["k.norm"] = TensorSpec((self.qk_dim,), "ones_plus_normal")
         if self.has_gate:
             specs["g"] = TensorSpec((self.heads if self.gate == "head" else self.a_dim, h))
+        if self.has_sink:
+            specs["sink"] = TensorSpec((self.heads,))
         if self.v_mix:
             specs["vmix"] = TensorSpec(())
         return specs
@@ -102,6 +110,8 @@ class GatedAttention(Mixer):
         if n % 8:                                 # the tensor-core projection wants output rows of whole 16 bytes
             rows.append(torch.zeros((8 - n % 8, rows[0].shape[1]), dtype=dt, device=rows[0].device))
         self.proj = Linear(torch.cat(rows, dim=0), self.rt)
+        if self.has_sink:
+            self.sink = tensors["sink"].to(torch.float32).contiguous()
         if self.v_mix == "mix":
             self.lam = float(tensors["vmix"])
         self.o = Linear(tensors["o"], self.rt)
@@ -140,7 +150,7 @@ class GatedAttention(Mixer):
         qkv = ws.take("attn.qkv", (T, (self.heads + 2 * self.kv_heads) * D), rt.dtype)
         B.qkv_prep(proj, self.bias, qkv, ctx.batch, kv, self.heads, self.qk_dim, self.v_dim, self.inv_freq, self.rotary_dim,
                    self.pairing, self.wq, self.wk, self.eps, writes_cache, rt.err, ctx.stream, rot_mul=self.rot_mul,
-                   v_first=v_first, lam=self.lam)
+                   v_first=v_first, lam=self.lam, temp_coef=self.temp_coef, temp_every=self.temp_every)
         out = ws.take("attn.out", (T, self.heads * D), rt.dtype)
         from_cache = ctx.kind == "decode" or not writes_cache
         if from_cache and ctx.kind == "prompt":
@@ -153,7 +163,7 @@ class GatedAttention(Mixer):
             from . import fast_attention
             done = fast_attention.apply(self, qkv, out, ctx, cache_view, from_cache)
         if not done:
-            B.attention_plain(qkv, out, ctx.batch, kv, self.heads, self.scale, from_cache, rt.err, ctx.stream)
+            B.attention_plain(qkv, out, ctx.batch, kv, self.heads, self.scale, from_cache, rt.err, ctx.stream, sink=self.sink)
         if self.has_gate or D != self.v_dim:
             gated = ws.take("gattn.gated", (T, self.a_dim), rt.dtype)
             B.gate_mul(out, proj[:, n_qkv:] if self.has_gate else None, gated, T, self.heads, D, self.v_dim, ctx.stream,

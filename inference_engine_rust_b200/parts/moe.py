@@ -19,6 +19,12 @@ their sum; with `score: "sigmoid"` every output is scored by its own sigmoid ins
 run's score is the sum of its two largest choice scores, and `route_scale` / `out_scale` multiply the weights; the last `identity` router outputs stand for experts without tensors that return their input; the
 experts' activation is any member of the gated-activation family (`activation`, `limit`), and they have no
 shared expert and no router bias.
+
+`UngatedMoE` (kind "ungated_moe") takes the same router, with weights that may be the chosen scores as they are
+(`renormalize: false`), and experts without a gate, W_down act(W_up h); a shared expert of the same form is multiplied by
+sigmoid(W_sg h), one number per token.  The up product's epilogue applies the activation and each token's weight of the
+expert that a column belongs to, so that nothing stands between the two products; W_sg is one more row of the router's
+product, and the routing kernel adds the identity experts' share itself.
 """
 from __future__ import annotations
 
@@ -26,6 +32,7 @@ from typing import Dict, Mapping
 
 import torch
 
+from ..config.specs import PartSpec
 from ..csrc import bindings as B
 from ..weights.loader import TensorSpec
 from .base import FeedForward, Runtime, StepContext, register_part
@@ -156,6 +163,15 @@ class GroupedMoE(MoE):
         wid = ws.take("moe.identity_share", (T,), torch.float32)
         idx = ws.take("moe.chosen", (T, self.top), torch.int32)
         w = ws.take("moe.chosen_weights", (T, self.top), torch.float32)
+        z, by_output = self._router_logits(xn, N, ctx)
+        B.router_grouped(z, self.correction, T, E, N, self.top, self.groups, self.keep, wt, wid, idx, w, ctx.stream,
+                         by_output=by_output, score=self.score, group_score=self.group_score, weight_eps=self.weight_eps,
+                         weight_scale=self.weight_scale)
+        return wt, (wid if self.identity else None)
+
+    def _router_logits(self, xn, N: int, ctx: StepContext):
+        """The fp32 product of the step's rows with the router's N rows, and whether it lies by output ([N, T]) or by token."""
+        ws, T = self.rt.workspace, ctx.n_tokens
         by_output = False
         if (self.rt.fast and T > SKINNY_ROUTER_MIN_TOKENS and N <= 32 and isinstance(xn, torch.Tensor)
                 and xn.dtype == torch.bfloat16 and self.router.weight.dtype == torch.bfloat16):
@@ -169,11 +185,61 @@ class GroupedMoE(MoE):
         if not by_output:
             z = ws.take("moe.logits", (T, N), torch.float32)
             self.router.apply(xn, z, T, ctx.stream)
-        B.router_grouped(z, self.correction, T, E, N, self.top, self.groups, self.keep, wt, wid, idx, w, ctx.stream,
+        return z, by_output
+
+
+class UngatedMoE(GroupedMoE):
+    graph_safe = True
+
+    def __init__(self, spec, rt: Runtime):
+        shared = int(spec["shared_ff"]) if spec.get("shared_ff") else 0
+        super().__init__(PartSpec(spec.kind, {**spec.params, "shared_ff": None, "activation": "silu"}), rt)
+        self.shared_ff = shared
+        self.inter = self.experts * self.expert_ff + shared
+        self.activation = spec.get("activation", "gelu")
+        self.renormalize = bool(spec.get("renormalize", True))
+        self.router_rows = self.outputs + (1 if shared else 0)
+        self.wt_cols = self.experts + (1 if shared else 0)
+        self.up = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        h, f, s = self.hidden_size, self.expert_ff, self.shared_ff
+        out = {"router": TensorSpec((self.outputs, h)), "correction": TensorSpec((self.outputs,))}
+        for e in range(self.experts):
+            out[f"e{e}.up"], out[f"e{e}.down"] = TensorSpec((f, h)), TensorSpec((h, f))
+        if s:
+            out["shared.up"], out["shared.down"], out["shared.sg"] = TensorSpec((s, h)), TensorSpec((h, s)), TensorSpec((1, h))
+        return out
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        dt = self.rt.dtype
+        names = [f"e{e}" for e in range(self.experts)] + (["shared"] if self.shared_ff else [])
+        self.up = Linear(torch.cat([tensors[f"{n}.up"].to(dt) for n in names], dim=0), self.rt)
+        self.down = Linear(torch.cat([tensors[f"{n}.down"].to(dt) for n in names], dim=1), self.rt)
+        rows = [tensors["router"].to(dt)] + ([tensors["shared.sg"].to(dt)] if self.shared_ff else [])
+        self.router = Linear(torch.cat(rows, dim=0), self.rt)
+        self.correction = tensors["correction"].to(torch.float32).contiguous()
+
+    def weight_bytes(self) -> int:
+        return self.up.nbytes() + self.down.nbytes() + self.router.nbytes()
+
+    def forward(self, xn, residual, ctx: StepContext) -> None:
+        rt, ws, T, E = self.rt, self.rt.workspace, ctx.n_tokens, self.experts
+        z, by_output = self._router_logits(xn, self.router_rows, ctx)
+        wt = ws.take("moe.weights", (T, self.wt_cols), torch.float32)
+        wid = ws.take("moe.identity_share", (T,), torch.float32)
+        idx = ws.take("moe.chosen", (T, self.top), torch.int32)
+        w = ws.take("moe.chosen_weights", (T, self.top), torch.float32)
+        B.router_grouped(z, self.correction, T, E, self.outputs, self.top, self.groups, self.keep, wt, wid, idx, w, ctx.stream,
                          by_output=by_output, score=self.score, group_score=self.group_score, weight_eps=self.weight_eps,
-                         weight_scale=self.weight_scale)
-        return wt, (wid if self.identity else None)
+                         weight_scale=self.weight_scale, renormalize=self.renormalize, shared_gate=bool(self.shared_ff),
+                         x=xn if self.identity else None, residual=residual if self.identity else None)
+        act = ws.take("ffn.act", (T, self.inter), rt.dtype)
+        self.up.apply(xn, act, T, ctx.stream, epilogue=B.epilogue(self.activation, scale=wt, blocks=E if self.shared_ff else E - 1,
+                                                                  block_cols=self.expert_ff))
+        self.down.apply(act, residual, T, ctx.stream, add_residual=True, ctx=ctx)
 
 
+register_part("ffn", "ungated_moe", UngatedMoE)
 register_part("ffn", "moe", MoE)
 register_part("ffn", "grouped_moe", GroupedMoE)

@@ -59,12 +59,25 @@ class RMSNorm(Norm):
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         w = tensors["weight"]
         self.weight = (w.to(torch.float32) + self.offset).contiguous() if self.offset else w.contiguous()
+        self._scaled = {}            # the fp32 weight times a factor, by factor
         self._weight_f32 = self.weight if self.weight.dtype == torch.float32 else self.weight.to(torch.float32)
 
-    def add_normed(self, y, x, cast, ctx, rows: int) -> None:
-        """x[:rows] += norm(y[:rows]) for a layer that norms a sublayer's output (fp32 both); clears y's rows
-        for the sublayer to come and writes the new rows into `cast` (the run's dtype, optional)."""
-        B.add_normed(x, y, self._weight_f32, cast, rows, self.eps, ctx.stream)
+    def add_normed(self, y, x, cast, ctx, rows: int, factor: float = 1.0, then: "RMSNorm" = None) -> None:
+        """x[:rows] += factor * norm(y[:rows]) for a layer that norms a sublayer's output (fp32 both); clears y's rows
+        for the sublayer to come and writes the new rows into `cast` (the run's dtype, optional), or their norm by `then`,
+        the norm in front of that sublayer."""
+        w = self._weight_f32
+        if factor != 1.0:
+            w = self._scaled.get(factor)
+            if w is None:
+                w = self._scaled[factor] = self._weight_f32 * factor
+        B.add_normed(x, y, w, cast, rows, self.eps, ctx.stream, w2=then._weight_f32 if then is not None else None,
+                     eps2=then.eps if then is not None else 0.0)
+
+    def begin_rows(self, x, out, ctx, rows: int, clear=None, e=None, step=None, keep=None) -> None:
+        """out[:rows] = norm(x) of rows that first become x + e + step (each optional; `keep` receives what they were);
+        clears `clear`'s rows for the sublayer to come."""
+        B.rows_begin(x, rows, ctx.stream, e=e, step=step, keep=keep, y=clear, out=out, w2=self._weight_f32, eps2=self.eps)
 
     def forward(self, x, out, ctx, rows_idx=None, rows=None) -> None:
         B.rmsnorm(x, self.weight, out, self.eps, ctx.stream, rows_idx=rows_idx, rows=rows)
