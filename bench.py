@@ -444,12 +444,12 @@ def main() -> int:
     ap.add_argument("--kernels", action="store_true",
                     help="also time the dominant kernels one by one with CUDA events (projections and decode "
                          "attention at the decode batch, projections at the prefill length): key 'kernels'")
-    ap.add_argument("--design", default=None, choices=["vefulix", "sifasun", "kuvelix", "vufinex", "botulorn"],
+    ap.add_argument("--design", default=None, choices=["vefulix", "sifasun", "kuvelix", "vufinex", "botulorn", "gidurax"],
                     help="instead of the default workload: prefill and decode of that design at Mistral 7B's width, "
                          "depth (--layers, default 8) and feed-forward size beside Mistral 7B itself, with a table of "
                          "each step's kernels against what their bytes and FLOPs allow (one JSON line)")
     ap.add_argument("--design-sizes", default="7b", choices=["7b", "12b"],
-                    help="with --design sifasun, kuvelix, vufinex or botulorn: the sizes of Mistral 7B (default) or of Mistral NeMo 12B")
+                    help="with --design sifasun, kuvelix, vufinex, botulorn or gidurax: the sizes of Mistral 7B (default) or of Mistral NeMo 12B")
     ap.add_argument("--design-beside", default="mistral", choices=["mistral", "vefulix"],
                     help="with --design: the model that runs beside it at equal sizes, Mistral (default) or, at the 7B "
                          "sizes, Vefulix (the other design with recurrences, latent attention and experts)")
@@ -457,8 +457,8 @@ def main() -> int:
 
     if a.design is not None and a.impl != "reference":
         from inference_engine_rust_b200 import bench_designs
-        if a.design_sizes == "12b" and a.design not in ("sifasun", "kuvelix", "vufinex", "botulorn"):
-            ap.error("--design-sizes 12b is there for --design sifasun, kuvelix, vufinex and botulorn only")
+        if a.design_sizes == "12b" and a.design not in ("sifasun", "kuvelix", "vufinex", "botulorn", "gidurax"):
+            ap.error("--design-sizes 12b is there for --design sifasun, kuvelix, vufinex, botulorn and gidurax only")
         if a.design_beside == "vefulix" and (a.design_sizes != "7b" or a.design == "vefulix"):
             ap.error("--design-beside vefulix is there for another design at the 7B sizes")
         base = "vefulix-7b-sizes" if a.design_beside == "vefulix" else "7b-v0.1" if a.design_sizes == "7b" else "nemo-12b"

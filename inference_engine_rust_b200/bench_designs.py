@@ -20,7 +20,8 @@ LAUNCHERS = ["embed_gather", "rmsnorm", "rope_kv_store", "silu_mul", "gemm_plain
              "mlstm_recur", "gated_head_norm", "latent_norm_store", "latent_attention_prompt", "latent_attention_decode_tc",
              "latent_attention_decode", "router_topk", "moe_scale", "add_normed", "cast_rows", "scale_values", "qk_prep",
              "rglru_conv", "rglru_gates", "rglru_scan", "qkv_prep", "gate_mul", "router_grouped", "gated_act_mul",
-             "token_shift", "wkv_decay", "wkv_recur", "wkv_finish", "latent_prep", "head_gate_mul", "layernorm", "embed_pairs"]
+             "token_shift", "wkv_decay", "wkv_recur", "wkv_finish", "latent_prep", "head_gate_mul", "layernorm", "embed_pairs",
+             "rows_begin", "selective_conv", "selective_scan", "epilogue_rows"]
 GEMMS = {"gemm_plain", "gemm_tc", "gemm_rows", "gemm_tc_scaled", "gemm_tc_gated", "gemm_tc_gated_scaled"}
 
 
@@ -237,6 +238,38 @@ def _costs(cfg: dict, T: int, n_seqs: int, ctx: int, prompt: bool) -> Dict[str, 
             out["latent_attention_decode"] = out["latent_attention_decode_tc"] = (
                 2.0 * n_seqs * m["heads"] * seen * (wide + m["kv_rank"]), True,
                 n_seqs * seen * wide * 2 + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"] * 2)
+    elif cfg.get("architecture") == "Gidurax":
+        H = cfg["width"]
+        out["rows_begin"] = out["add_normed"] = (0.0, False, T * H * 18)           # y and x read and written, the normed row written
+        out["rmsnorm"] = (0.0, False, T * H * 6)
+        by = {l["type"]: l["mixer"] for l in cfg["layers"]}
+        if "mamba1" in by:
+            m = by["mamba1"]
+            C, N = m["inner"], m["state"]
+            out["selective_conv"] = (0.0, False, T * C * 4)
+            # dt, u and z read, the result written, the state of every sequence read and written; 6 FLOPs per state and token
+            out["selective_scan"] = (6.0 * T * C * N, False, T * (C * 10 + 4 * N) + 2 * 4 * n_seqs * C * N)
+        if "delta" in by:
+            m = by["delta"]
+            C = 2 * m["kv_heads"] * m["dim"] + m["heads"] * m["vdim"]
+            state = 2 * 4 * n_seqs * m["heads"] * m["dim"] * m["vdim"]
+            out["delta_prep"] = (0.0, False, T * C * 6)
+            out["delta_recur"] = (8.0 * T * m["heads"] * m["dim"] * m["vdim"], False, T * (C + m["heads"] * m["vdim"]) * 4 + state)
+            out["gated_head_norm"] = (0.0, False, T * m["heads"] * m["vdim"] * 8)
+        if "attention" in by:
+            m = by["attention"]
+            D = -(-max(m["dim"], m["vdim"]) // 16) * 16
+            qd, kd, vd = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+            packed = (m["heads"] + 2 * m["kv_heads"]) * D
+            out["qkv_prep"] = (0.0, False, T * ((qd + kd + vd) * 4 + packed * 2 + 2 * m["kv_heads"] * D * 2))
+            if prompt:
+                out[f"attention_prefill [head {D}]"] = (4.0 * m["heads"] * D * T * (T + 1) / 2, True,
+                                                        T * (2 * m["heads"] * D + 2 * m["kv_heads"] * D) * 2)
+            out["attention_decode_tc"] = (0.0, False, n_seqs * ctx * 2 * m["kv_heads"] * D * 2)
+        mlp = next((l["mlp"] for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe"), None)
+        if mlp:
+            r = mlp["router"]
+            out["router_grouped"] = (0.0, False, T * ((r["experts"] + r.get("identity", 0)) * 8 + (10 * H if r.get("identity") else 0)))
     else:
         hd = cfg["num_attention_heads"] * cfg["head_dim"]
         kvd = cfg["num_key_value_heads"] * cfg["head_dim"]

@@ -62,24 +62,21 @@ class GatedAct(Structure):
     _fields_ = [("g_max", c_float), ("u_max", c_float), ("u_bias", c_float), ("a", c_float), ("b", c_float)]
 
 
-ACT_NONE, ACT_GELU, ACT_SOFTPLUS = 0, 1, 2
-PLAIN_ACTIVATIONS = {"none": ACT_NONE, "gelu": ACT_GELU, "softplus": ACT_SOFTPLUS}     # "gelu": the exact (erf) form
+PLAIN_ACTIVATIONS = {"none": 0, "gelu": 1}     # "gelu": the exact (erf) form
 
 
 class Epilogue(Structure):
-    """Mirror of `IertEpilogue` (common.cuh): v <- act(v + bias[n]) * scale[t, min(n / block_cols, blocks)]."""
-    _fields_ = [("act", c_int), ("bias", c_void_p), ("scale", c_void_p), ("ld_scale", c_longlong), ("blocks", c_int),
-                ("block_cols", c_int)]
+    """Mirror of `IertEpilogue` (common.cuh): v <- act(v) * scale[t, min(n / block_cols, blocks)]."""
+    _fields_ = [("act", c_int), ("scale", c_void_p), ("ld_scale", c_longlong), ("blocks", c_int), ("block_cols", c_int)]
 
 
-def epilogue(act: str = "none", bias=None, scale=None, blocks: int = 0, block_cols: int = 1) -> Epilogue:
-    """What a projection does to each output before it stores it: `bias` fp32 [N], an activation by name, and a factor per
-    token and block of columns (`scale` fp32 [tokens, > blocks]: `blocks` blocks of `block_cols` columns, the rest one more)."""
+def epilogue(act: str = "none", scale=None, blocks: int = 0, block_cols: int = 1) -> Epilogue:
+    """What a projection does to each output before it stores it: an activation by name, and a factor per token and block
+    of columns (`scale` fp32 [tokens, > blocks]: `blocks` blocks of `block_cols` columns, the rest one more)."""
     if act not in PLAIN_ACTIVATIONS:
         raise KernelError(f"activation must be one of {sorted(PLAIN_ACTIVATIONS)}, got {act!r}")
-    return Epilogue(act=PLAIN_ACTIVATIONS[act], bias=bias.data_ptr() if bias is not None else None,
-                    scale=scale.data_ptr() if scale is not None else None, ld_scale=scale.stride(0) if scale is not None else 0,
-                    blocks=blocks, block_cols=block_cols)
+    return Epilogue(act=PLAIN_ACTIVATIONS[act], scale=scale.data_ptr() if scale is not None else None,
+                    ld_scale=scale.stride(0) if scale is not None else 0, blocks=blocks, block_cols=block_cols)
 
 
 def gated_act(name: str, limit: Optional[float] = None) -> Optional[GatedAct]:
@@ -182,7 +179,7 @@ def _declare(lib) -> None:
         "iert_add_normed": [P, P, P, P, c_int, c_int, c_int, c_float, P, c_float, S],
         "iert_rows_begin": [P, P, P, P, P, P, c_int, c_int, c_int, P, c_float, S],
         "iert_selective_conv": [P, c_int, LL, P, P, P, LL, LL, P, c_int, c_int, POINTER(BatchView), S],
-        "iert_selective_scan": [P, c_int, P, P, LL, P, LL, P, P, P, LL, LL, P, c_int, c_int, c_int, POINTER(BatchView), S],
+        "iert_selective_scan": [P, c_int, P, P, P, LL, P, LL, P, P, P, LL, LL, P, c_int, c_int, c_int, POINTER(BatchView), S],
         "iert_cast_rows": [P, P, P, c_int, LL, S],
         "iert_scale_values": [P, LL, c_float, S],
         "iert_qk_prep": [P, LL, P, c_int, POINTER(BatchView), POINTER(KvView), c_int, P, c_int, c_int, P, P, c_float, c_float,
@@ -986,10 +983,10 @@ def selective_conv(x, taps, bias, state, ring_off: int, u, C: int, K: int, batch
                                      state.stride(0), ring_off, u.data_ptr(), C, K, byref(batch), stream), "selective_conv")
 
 
-def selective_scan(u, dt, bc, z, A2, D, state, s_off: int, out, C: int, N: int, one_token: bool, batch: BatchView, stream) -> None:
-    """S[c, n] <- exp(dt A) S + dt u B; out = (sum_n S C + D u) * silu(z) over the step's tokens; `bc`: rows that begin with
+def selective_scan(u, dt, dt_bias, bc, z, A2, D, state, s_off: int, out, C: int, N: int, one_token: bool, batch: BatchView, stream) -> None:
+    """S[c, n] <- exp(d A) S + d u B with d = softplus(dt + dt_bias); out = (sum_n S C + D u) * silu(z) over the step's tokens; `bc`: rows that begin with
     [B | C], `z`: rows of C numbers (both views that may be strided, in u's dtype), dt fp32 [T, C], A2 = A log2(e) (u fp32: A) fp32 [C, N],
     S [C, N] per slot in `state` at s_off."""
-    check(core().iert_selective_scan(u.data_ptr(), dtype_code(u.dtype), dt.data_ptr(), bc.data_ptr(), bc.stride(0), z.data_ptr(),
+    check(core().iert_selective_scan(u.data_ptr(), dtype_code(u.dtype), dt.data_ptr(), dt_bias.data_ptr(), bc.data_ptr(), bc.stride(0), z.data_ptr(),
                                      z.stride(0), A2.data_ptr(), D.data_ptr(), state.data_ptr(), state.stride(0), s_off,
                                      out.data_ptr(), C, N, 1 if one_token else 0, byref(batch), stream), "selective_scan")

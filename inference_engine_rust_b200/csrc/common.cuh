@@ -146,14 +146,12 @@ struct IertGatedAct {
 };
 
 // What a projection that stores its outputs may do to each output v[t, n] before it is rounded:
-//   v <- v + bias[n];   v <- act(v);   v <- v * scale[t * ld_scale + min(n / block_cols, blocks)]
-// act: 0 none; 1 the exact GELU, v (1 + erf(v / sqrt 2)) / 2; 2 softplus.  The column scale serves experts whose matrices
-// are stacked by rows: `blocks` runs of block_cols columns, and whatever follows them (an expert every token uses) is one
-// more block.
-enum : int { IERT_ACT_NONE = 0, IERT_ACT_GELU = 1, IERT_ACT_SOFTPLUS = 2 };
+//   v <- act(v);   v <- v * scale[t * ld_scale + min(n / block_cols, blocks)]
+// act: 0 none; 1 the exact GELU, v (1 + erf(v / sqrt 2)) / 2.  The column scale serves experts whose matrices are stacked by
+// rows: `blocks` runs of block_cols columns, and whatever follows them (an expert every token uses) is one more block.
+enum : int { IERT_ACT_NONE = 0, IERT_ACT_GELU = 1 };
 struct IertEpilogue {
   int act;
-  const float* bias;       // fp32 [N], or null
   const float* scale;      // fp32, or null
   long long ld_scale;
   int blocks, block_cols;
@@ -161,28 +159,21 @@ struct IertEpilogue {
 
 namespace iert {
 
-__device__ __forceinline__ bool epilogue_on(const IertEpilogue& e) { return e.act != IERT_ACT_NONE || e.bias || e.scale; }
-__device__ __forceinline__ float epilogue_act(float v, int act) {
-  if (act == IERT_ACT_GELU) return 0.5f * v * (1.0f + erff(v * 0.70710678f));
-  if (act == IERT_ACT_SOFTPLUS) return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));
-  return v;
-}
+__device__ __forceinline__ bool epilogue_on(const IertEpilogue& e) { return e.act != IERT_ACT_NONE || e.scale; }
+__device__ __forceinline__ float gelu_exact(float v) { return 0.5f * v * (1.0f + erff(v * 0.70710678f)); }
 __device__ __forceinline__ int epilogue_block(int n, const IertEpilogue& e) { return min(n / e.block_cols, e.blocks); }
 __device__ __forceinline__ float epilogue_value(float v, int t, int n, const IertEpilogue& e) {
-  if (e.bias) v += e.bias[n];
-  v = epilogue_act(v, e.act);
+  if (e.act == IERT_ACT_GELU) v = gelu_exact(v);
   if (e.scale) v *= e.scale[(long long)t * e.ld_scale + epilogue_block(n, e)];
   return v;
 }
-// N consecutive outputs of one token from column n on (those beyond n_end are left alone).
+// N consecutive outputs of one token from column n on (columns that the matrix does not have are nobody's).
 template <int N>
-__device__ __forceinline__ void epilogue_run(float* v, int t, int n, int n_end, const IertEpilogue& e) {
-  if (e.bias) {
+__device__ __forceinline__ void epilogue_run(float* v, int t, int n, const IertEpilogue& e) {
+  if (e.act == IERT_ACT_GELU) {
 #pragma unroll
-    for (int j = 0; j < N; ++j) if (n + j < n_end) v[j] += e.bias[n + j];
+    for (int j = 0; j < N; ++j) v[j] = gelu_exact(v[j]);
   }
-#pragma unroll
-  for (int j = 0; j < N; ++j) v[j] = epilogue_act(v[j], e.act);
   if (e.scale) {
     const float* row = e.scale + (long long)t * e.ld_scale;
     const int b0 = epilogue_block(n, e), b1 = epilogue_block(n + N - 1, e);

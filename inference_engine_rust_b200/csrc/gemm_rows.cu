@@ -71,7 +71,7 @@ struct RowsParams {
   int* err;
   IertRowScale scale;                     // scale.sumsq != null: the outputs are multiplied by the rows' 1 / rms
   IertNormAhead ahead;                    // ahead.scaled_out != null (residual add): the next norm's first half
-  IertEpilogue ep;                        // mode 0: bias, activation and column scale of the outputs (see common.cuh)
+  IertEpilogue ep;                        // mode 0: activation and column scale of the outputs (see common.cuh)
   int trace_seq;
   int w_dynamic;                          // the matrix operand was written by the kernel in front: nothing is fetched before the wait
 };
@@ -334,7 +334,7 @@ IERT_API int iert_gemm_rows_trace_read(unsigned long long* stamps, int* meta) {
 // IERT_BAD_ARGUMENT is returned and nothing is launched.  force_stages: 0 = choose.
 //   scale (optional)  the rows of x are the first half of an RMSNorm (IertNormAhead of the kernel that
 //                     wrote them): the outputs are multiplied by each row's 1 / rms (see common.cuh).
-//   ep (optional; mode 0)  bias, activation and column scale of the outputs (after `scale`).
+//   ep (optional; mode 0)  activation and column scale of the outputs (after `scale`).
 //   w_dynamic         w is no stored weight but rows that the kernel in front wrote (a few stored rows against many
 //                     tokens, the tokens as the streamed matrix): it is not fetched ahead of the dependency wait.
 //   ahead (optional; mode 1)  the first half of the NEXT norm over the new rows of `out`: ahead->parts
@@ -361,7 +361,7 @@ IERT_API int iert_gemm_rows(const void* x, long long ldx, const void* w, long lo
   p.scale = IertRowScale{nullptr, 0, 0, 0.f};
   if (scale) p.scale = *scale;
   p.ahead = IertNormAhead{nullptr, 0, nullptr, 0, nullptr, 0};
-  p.ep = ep ? *ep : IertEpilogue{IERT_ACT_NONE, nullptr, nullptr, 0, 0, 1};
+  p.ep = ep ? *ep : IertEpilogue{IERT_ACT_NONE, nullptr, 0, 0, 1};
   p.kb_total = (K + KB - 1) / KB;
   p.n_stages = (p.kb_total + KPS - 1) / KPS;
   const int stage_bytes = KPS * (W_BYTES + nt * 8 * KB * 2);

@@ -83,7 +83,7 @@ struct GemmParams {
                         // the rows' 1 / rms
   IertNormAhead ahead;  // split-K residual add, tiles of 32 or 64 tokens: ahead.scaled_out != null: the reduction also
                         // writes the next norm's first half
-  IertEpilogue ep;      // plain stores: bias, activation and column scale of every output (see common.cuh)
+  IertEpilogue ep;      // plain stores: activation and column scale of every output (see common.cuh)
   IertGatedAct act;     // gated launches: the activation (see common.cuh)
   int trace_seq;        // >= 0: the launch's row in the trace (builds with IERT_GEMM_TRACE only)
   uint32_t poll_limit;  // polls of a tile's counter before a CTA gives up waiting for the other CTAs of its tile
@@ -127,7 +127,7 @@ __device__ __forceinline__ void write_out_any(const GemmParams& p, int tok, int 
 
 // Four consecutive outputs of one token, vectorised when aligned and inside the matrix.
 __device__ __forceinline__ void write_out4(const GemmParams& p, int tok, int n, float4 r) {
-  if (p.mode == MODE_STORE && epilogue_on(p.ep)) epilogue_run<4>(reinterpret_cast<float*>(&r), tok, n, p.N, p.ep);
+  if (p.mode == MODE_STORE && epilogue_on(p.ep)) epilogue_run<4>(reinterpret_cast<float*>(&r), tok, n, p.ep);
   const bool whole = n + 4 <= p.N && (p.ldo & 3) == 0 && ((uintptr_t)p.out & 15) == 0;
   if (whole && p.out_dtype == IERT_F32) {
     float4* o = reinterpret_cast<float4*>((float*)p.out + (long long)tok * p.ldo + n);
@@ -513,7 +513,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
           float v[16];
           tmem_ld16(taddr + c, v);
           if (tok >= p.M) continue;
-          if (p.mode == MODE_STORE && epilogue_on(p.ep)) epilogue_run<16>(v, tok, n0 + c, p.N, p.ep);
+          if (p.mode == MODE_STORE && epilogue_on(p.ep)) epilogue_run<16>(v, tok, n0 + c, p.ep);
           const bool full16 = n0 + c + 16 <= p.N;
           if (p.out_dtype == IERT_F32) {
             float* o = (float*)p.out + (long long)tok * p.ldo + n0 + c;
@@ -977,7 +977,7 @@ IERT_API int iert_gemm_tc_counter_count() { return 8192; }
 // x: [M, K] bf16, row stride ldx; w: [N, K] bf16, row stride ldw; out: [M, N] of out_dtype, row
 // stride ldo.  mode 0 stores, mode 1 adds into out.  K, ldx and ldw must be multiples of 8
 // and the pointers 16-byte aligned (TMA); otherwise IERT_BAD_ARGUMENT is returned and nothing
-// is launched.  ep (optional, mode 0): bias, activation and column scale of the outputs.  ws / counters: scratch for split-K, shared by all launches on one stream;
+// is launched.  ep (optional, mode 0): activation and column scale of the outputs.  ws / counters: scratch for split-K, shared by all launches on one stream;
 // counters must be zero before the first launch.  force_*: 0 = choose.
 namespace {
 int gemm_tc_impl(const void* x, long long ldx, const void* w, long long ldw, void* out, int out_dtype,
@@ -1013,7 +1013,7 @@ int gemm_tc_impl(const void* x, long long ldx, const void* w, long long ldw, voi
   p.scale = IertRowScale{nullptr, 0, 0, 0.f};
   p.ahead = IertNormAhead{nullptr, 0, nullptr, 0, nullptr, 0};
   if (scale) p.scale = *scale;
-  p.ep = ep ? *ep : IertEpilogue{IERT_ACT_NONE, nullptr, nullptr, 0, 0, 1};
+  p.ep = ep ? *ep : IertEpilogue{IERT_ACT_NONE, nullptr, 0, 0, 1};
   p.tail_parts = 1; p.full_tiles = 0; p.tma_out = 0; p.t_group = 1 << 30;
   p.out = out; p.ldo = ldo; p.out_dtype = out_dtype; p.mode = mode;
   p.M = M; p.N = N; p.K = K;
@@ -1194,7 +1194,7 @@ int gemm_tc_gated_impl(const void* x, long long ldx, const void* w, long long ld
   if (scale && (!scale->sumsq || scale->parts <= 0 || scale->hidden <= 0)) return IERT_BAD_ARGUMENT;
   GemmParams p;
   p.scale = IertRowScale{nullptr, 0, 0, 0.f};
-  p.ep = IertEpilogue{IERT_ACT_NONE, nullptr, nullptr, 0, 0, 1};
+  p.ep = IertEpilogue{IERT_ACT_NONE, nullptr, 0, 0, 1};
   p.tail_parts = 1; p.full_tiles = 0; p.tma_out = 0; p.t_group = 1 << 30;
   p.out = act; p.ldo = ldo; p.out_dtype = IERT_BF16; p.mode = MODE_GATED_SILU;
   p.act = fn ? *fn : IertGatedAct{INFINITY, INFINITY, 0.f, 1.f, 0.f};

@@ -67,7 +67,7 @@ class GatedDelta(Mixer):
 
     def load(self, t: Mapping[str, torch.Tensor]) -> None:
         self.proj = Linear(_stack(self.rt, [t["q"], t["k"], t["v"], t["g"]]), self.rt)
-        self.gates = Linear(_stack(self.rt, [t["b"], t["a"]], 4), self.rt)
+        self.gates = Linear(_stack(self.rt, [t["b"], t["a"]], 4), self.rt, narrow=True)
         self.conv_w = _f32(torch.cat([t["q.conv"], t["k.conv"], t["v.conv"]], dim=0))
         self.A_log, self.dt_bias, self.norm = _f32(t["A_log"]), _f32(t["dt_bias"]), _f32(t["norm"])
         self.o = Linear(t["o"], self.rt)

@@ -12,8 +12,8 @@ mixer's input, C = `inner` channels, N = `state` numbers kept per channel, R = `
 State per sequence (fp32, zero at the start, carried from step to step): S and the convolution's last inputs.  Tensors: in
 [2C, hidden], conv [C, taps], conv.b [C], x [R + 2N, C], dt [C, R], dt.b [C], A_log [C, N], D [C], o [hidden, C].
 
-The products run in the run's dtype; the step sizes leave theirs in fp32 with bias and softplus applied by the product's
-epilogue; convolution and scan are the kernels of `csrc/selective_scan.cu` (fp32 arithmetic and state)."""
+The products run in the run's dtype, W_dt's with fp32 outputs; bias, softplus and everything after are fp32 arithmetic in the
+kernels of `csrc/selective_scan.cu`."""
 from __future__ import annotations
 
 import math
@@ -85,9 +85,9 @@ class SelectiveScan(Mixer):
         p = ws.take("scan.p", (T, self.p_width), rt.dtype)
         self.x.apply(u, p, T, ctx.stream)
         dt = ws.take("scan.dt", (T, C), torch.float32)
-        self.dt.apply(p[:, :self.R_pad], dt, T, ctx.stream, epilogue=B.epilogue("softplus", bias=self.dt_b))
+        self.dt.apply(p[:, :self.R_pad], dt, T, ctx.stream)
         out = ws.take("scan.out", (T, C), rt.dtype)
-        B.selective_scan(u, dt, p[:, self.R_pad:], xz[:, C:], self.A2, self.D, state, 0, out, C, self.N, ctx.kind == "decode",
+        B.selective_scan(u, dt, self.dt_b, p[:, self.R_pad:], xz[:, C:], self.A2, self.D, state, 0, out, C, self.N, ctx.kind == "decode",
                          ctx.batch, ctx.stream)
         self.o.apply(out, residual, T, ctx.stream, add_residual=True, ctx=ctx)
 
