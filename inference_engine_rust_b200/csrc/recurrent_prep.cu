@@ -47,6 +47,16 @@ struct DeltaPrepArgs {
   int G, D, H, V, taps;
 };
 
+// beta and decay of a token's heads, by one warp
+__device__ __forceinline__ void write_gates(const DeltaPrepArgs& a, int t, int lane) {
+  for (int h = lane; h < a.H; h += 32) {
+    const float gb = a.gates[(size_t)t * a.gld + h], ga = a.gates[(size_t)t * a.gld + a.H + h];
+    a.beta[(size_t)t * a.H + h] = sigmoid_f(gb);
+    // 1 + expm1: a decay near 1 keeps its distance from 1, whose error a long sequence would gather
+    a.decay[(size_t)t * a.H + h] = 1.0f + expm1f(-expf(a.A_log[h]) * softplus_f(ga + a.dt_bias[h]));
+  }
+}
+
 // One warp per (token, unit), a unit being a q head, a k head or a v head: a lane has a few channels, all its
 // loads are independent, and the unit norm is a warp sum: no shared memory, no block barrier, and a step
 // of a handful of tokens still spreads over the device.  A block is four tokens of one unit.
@@ -102,13 +112,96 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(DeltaPrepArgs a, IertBa
     const int i = lane + 32 * k;
     if (i < n) a.qkv[(size_t)t * C + c0 + i] = val[k] * f;
   }
-  if (unit == 0)
-    for (int h = lane; h < a.H; h += 32) {
-      const float gb = a.gates[(size_t)t * a.gld + h], ga = a.gates[(size_t)t * a.gld + a.H + h];
-      a.beta[(size_t)t * a.H + h] = sigmoid_f(gb);
-      // 1 + expm1: a decay near 1 keeps its distance from 1, whose error a long sequence would gather
-      a.decay[(size_t)t * a.H + h] = 1.0f + expm1f(-expf(a.A_log[h]) * softplus_f(ga + a.dt_bias[h]));
+  if (unit == 0) write_gates(a, t, lane);
+}
+
+// The same for unit sizes in whole groups of four up to 128 (a lane holds four channels) and TAPS known: a warp takes PER
+// consecutive tokens of one unit, whose inputs (neighbours in memory, whatever sequences they belong to) are all asked for before
+// the first is used; the last inputs and the taps stay in registers from token to token.
+template <typename T> struct Four;
+template <> struct Four<float> { typedef float4 raw; };
+template <> struct Four<__nv_bfloat16> { typedef uint2 raw; };
+__device__ __forceinline__ float4 four(const float4& r) { return r; }
+__device__ __forceinline__ float4 four(const uint2& r) {
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
+template <typename T, int TAPS, int PER>
+__global__ void __launch_bounds__(128) delta_prep_vec_kernel(DeltaPrepArgs a, IertBatchView b) {
+  typedef typename Four<T>::raw Raw;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t0 = (blockIdx.x * 4 + warp) * PER, unit = blockIdx.y;
+  if (t0 >= b.n_tokens) return;
+  const int GD = a.G * a.D, C = 2 * GD + a.H * a.V;
+  const bool is_v = unit >= 2 * a.G;
+  const int c0 = is_v ? 2 * GD + (unit - 2 * a.G) * a.V : unit * a.D;
+  const int n = is_v ? a.V : a.D;
+  const bool mine = 4 * lane < n;
+  const int c = c0 + (mine ? 4 * lane : 0);
+  float4 w[TAPS], hist[TAPS];                      // w[j], hist[j]: tap and input j tokens back
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+    const float* wp = a.conv_w + (size_t)c * TAPS + (TAPS - 1 - j);
+    w[j] = make_float4(wp[0], wp[TAPS], wp[2 * TAPS], wp[3 * TAPS]);
+  }
+  pdl_wait();
+  const T* proj = (const T*)a.proj;
+  Raw run[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i)
+    if (t0 + i < b.n_tokens) run[i] = *reinterpret_cast<const Raw*>(proj + (size_t)(t0 + i) * a.ld + c);
+  int slot = -1, q_begin = 0, q_end = 0, pos0 = 0;
+  bool known = false;
+  float* ring = nullptr;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int t = t0 + i;
+    if (t >= b.n_tokens) break;
+    bool fresh = false;
+    if (!known || t >= q_end) {                    // another sequence (or padding) from here on
+      const int s = sequence_of_token(b, t);
+      slot = s < 0 ? -1 : b.slot_ids[s];
+      known = slot >= 0;
+      if (known) {
+        q_begin = b.cu_q[s];
+        q_end = b.cu_q[s + 1];
+        pos0 = b.pos0[s];
+        ring = a.state + (size_t)slot * a.state_stride + a.conv_off;
+        fresh = true;
+      }
     }
+    if (slot < 0) continue;
+    const int pos = pos0 + (t - q_begin);
+    if (fresh) {
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j) {
+        if (t - j >= q_begin) hist[j] = four(*reinterpret_cast<const Raw*>(proj + (size_t)(t - j) * a.ld + c));
+        else if (pos - j >= 0) hist[j] = *reinterpret_cast<const float4*>(ring + (size_t)((pos - j) % TAPS) * C + c);
+        else hist[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    }
+    hist[0] = four(run[i]);
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = TAPS - 1; j >= 0; --j) {          // oldest first
+      acc.x = fmaf(w[j].x, hist[j].x, acc.x); acc.y = fmaf(w[j].y, hist[j].y, acc.y);
+      acc.z = fmaf(w[j].z, hist[j].z, acc.z); acc.w = fmaf(w[j].w, hist[j].w, acc.w);
+    }
+    if (mine && t >= q_end - TAPS) *reinterpret_cast<float4*>(ring + (size_t)(pos % TAPS) * C + c) = hist[0];
+#pragma unroll
+    for (int j = TAPS - 1; j > 0; --j) hist[j] = hist[j - 1];
+    acc = make_float4(silu_f(acc.x), silu_f(acc.y), silu_f(acc.z), silu_f(acc.w));
+    float f = 1.f;
+    if (!is_v) {
+      const float ss = mine ? acc.x * acc.x + acc.y * acc.y + acc.z * acc.z + acc.w * acc.w : 0.f;
+      f = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
+      if (unit < a.G) f *= 1.0f / sqrtf((float)a.D);
+    }
+    if (mine) *reinterpret_cast<float4*>(a.qkv + (size_t)t * C + c) = make_float4(acc.x * f, acc.y * f, acc.z * f, acc.w * f);
+    if (unit == 0) write_gates(a, t, lane);
+  }
 }
 
 // o [T, H*V] fp32; gate: column gate_off + h*V + e of the packed projection; weight index
@@ -385,8 +478,22 @@ IERT_API int iert_delta_prep(const void* proj, int dtype, long long ld, const fl
     return IERT_BAD_ARGUMENT;
   DeltaPrepArgs a = {proj, ld, gates, gld, conv_w, A_log, dt_bias, state, state_stride, conv_off, qkv, beta, decay,
                      G, D, H, V, taps};
-  (void)C;
   const size_t smem = 0;
+  // groups of four channels, aligned in the projection, the state's ring and the result
+  const int elt = dtype == IERT_F32 ? 4 : 2;
+  if ((taps == 4 || taps == 3 || taps == 2) && D % 4 == 0 && V % 4 == 0 && D <= 128 && V <= 128 && ld % 4 == 0 && state_stride % 4 == 0 &&
+      conv_off % 4 == 0 && C % 4 == 0 && (((uintptr_t)state | (uintptr_t)qkv) & 15) == 0 && ((uintptr_t)proj % (4 * elt)) == 0 &&
+      (dtype == IERT_F32 || dtype == IERT_BF16)) {
+    const int per = batch->n_tokens >= 256 ? 8 : 1;
+    const dim3 vgrid((batch->n_tokens + 4 * per - 1) / (4 * per), 2 * G + H);
+#define VEC(T, K) do { if (per == 8) launch_dep(delta_prep_vec_kernel<T, K, 8>, vgrid, dim3(128), 0, stream, a, *batch); \
+                       else launch_dep(delta_prep_vec_kernel<T, K, 1>, vgrid, dim3(128), 0, stream, a, *batch); } while (0)
+#define BY_TAPS(T) do { if (taps == 4) VEC(T, 4); else if (taps == 3) VEC(T, 3); else VEC(T, 2); } while (0)
+    if (dtype == IERT_F32) BY_TAPS(float); else BY_TAPS(__nv_bfloat16);
+#undef BY_TAPS
+#undef VEC
+    return iert_check_launch("delta_prep");
+  }
   const dim3 grid((batch->n_tokens + 3) / 4, 2 * G + H);
   if (dtype == IERT_F32) launch_dep(delta_prep_kernel<float>, grid, dim3(128), smem, stream, a, *batch);
   else if (dtype == IERT_BF16) launch_dep(delta_prep_kernel<__nv_bfloat16>, grid, dim3(128), smem, stream, a, *batch);
