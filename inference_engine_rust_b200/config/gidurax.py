@@ -204,7 +204,7 @@ def build_spec(cfg: GiduraxConfig) -> ModelSpec:
     mamba1: in, conv, conv.b, x, dt, dt.b, A_log, D, o), `l<i>.mlp.{up,down}` or `l<i>.mlp.e<j>.{up,down}` with `l<i>.mlp.router`,
     `l<i>.mlp.correction` and `l<i>.mlp.shared.{up,down,sg}`; i is the layer's place in config.json."""
     norm = PartSpec("rmsnorm", {"eps": cfg.eps})
-    block = PartSpec("sandwich", {"factor": cfg.residual_mult})
+    block = PartSpec("sandwich_norm", {"factor": cfg.residual_mult})
     layers = []
     for i, layer in enumerate(cfg.layers):
         p = f"l{i}."

@@ -7,7 +7,7 @@ recurrence with a short convolution) and "parallel" (two mixers side by side); b
 both sublayers), mixer "gated_attention" (biases, a norm per head of q and k, a value size of its own, a sigmoid gate on
 the heads), ffn "grouped_moe" (scores over all outputs or a sigmoid each, choice inside the best groups, experts that return
 their input); mixer "wkv" (a matrix state with a decay per key channel, token shift); "tied_kv_attention" also takes a mask of
-chunks, "latent_attention" also a rotated key part shared by the heads and a gate per head; block "sandwich" (a norm on both sides
+chunks, "latent_attention" also a rotated key part shared by the heads and a gate per head; block "sandwich_norm" (a norm on both sides
 of each sublayer), mixer "selective_scan" (Mamba), ffn "mlp" (no gate) and "ungated_moe" (experts without a gate, a gated shared
 expert), pass "step_vectors" (what precedes each pass of a repeated run of layers)."""
 from .base import (Block, FeedForward, Head, Mixer, Norm, Part, PassStart, PositionEncoding, Runtime, StepContext, StepInput,

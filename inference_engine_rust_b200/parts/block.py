@@ -1,6 +1,6 @@
 """Arrangement of a layer's parts.  "two_norms": x += mixer(norm1(x)) + ffn(norm2(x)), both norms of the same
 x.  "shared_norm": h = norm1(x); x += mixer(h) + ffn(h) (one norm, read by both
-sublayers).  "sandwich": a norm on both sides of each
+sublayers).  "sandwich_norm": a norm on both sides of each
 sublayer.  "prenorm": x += mixer(norm1(x)); x += ffn(norm2(x)) (the second
 half left out for a layer without a feed-forward)
 (src/layers/block.rs:19-24,63-65; the residual uses the un-normed input,
@@ -184,10 +184,10 @@ class SandwichBlock(Block):
         self.post1, self.post2 = extra_norms["mixer_out"], extra_norms.get("ffn_out")
         self.factor = float(layer_spec.block.get("factor", 1.0))
         if ffn is not None and (norm2 is None or self.post2 is None):
-            raise ValueError("block 'sandwich' with a feed-forward needs a second norm and an extra norm 'ffn_out'")
+            raise ValueError("block 'sandwich_norm' with a feed-forward needs a second norm and an extra norm 'ffn_out'")
         for n in (norm1, norm2, self.post1, self.post2):
             if n is not None and not hasattr(n, "begin_rows"):
-                raise ValueError(f"block 'sandwich' needs norms with add_normed and begin_rows, got {type(n).__name__}")
+                raise ValueError(f"block 'sandwich_norm' needs norms with add_normed and begin_rows, got {type(n).__name__}")
 
     def _buffers(self, x):
         ws = self.rt.workspace
@@ -290,5 +290,5 @@ register_part("block", "prenorm", PreNormBlock)
 register_part("block", "two_norms", TwoNormsBlock)
 register_part("block", "shared_norm", SharedNormBlock)
 register_part("block", "outnorm", OutputNormBlock)
-register_part("block", "sandwich", SandwichBlock)
+register_part("block", "sandwich_norm", SandwichBlock)
 register_part("block", "hyper", HyperConnectionBlock)

@@ -39,7 +39,7 @@ def test_spec_of_a_configuration():
     assert [(e.layer, e.pass_start) for e in spec.schedule] == [(0, None), (1, 0), (2, None), (1, 1), (2, None), (1, 2), (2, None), (3, None)]
     assert spec.embedding_scale == 3.0 and spec.lm_head_name == "head" and spec.final_norm["eps"] == 1e-5
     assert spec.passes[0].kind == "step_vectors" and spec.passes[0]["times"] == 3 and spec.passes[1] == "loop."
-    assert all(l.block.kind == "sandwich" and l.block["factor"] == 0.6 for l in spec.layers)
+    assert all(l.block.kind == "sandwich_norm" and l.block["factor"] == 0.6 for l in spec.layers)
     a = spec.layers[0].mixer
     assert a.kind == "gated_attention" and a["sink"] and not a["bias"] and not a["gate"] and a["qk_norm"] == "head" and a["window"] is None
     assert a["q_temp"] == {"coef": 0.3, "every": 7.0} and (a["head_dim"], a["v_dim"], a["scale"]) == (10, 14, 0.4)
