@@ -240,7 +240,8 @@ def _costs(cfg: dict, T: int, n_seqs: int, ctx: int, prompt: bool) -> Dict[str, 
                 n_seqs * seen * wide * 2 + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"] * 2)
     elif cfg.get("architecture") == "Gidurax":
         H = cfg["width"]
-        out["rows_begin"] = out["add_normed"] = (0.0, False, T * H * 18)           # y and x read and written, the normed row written
+        out["add_normed"] = (0.0, False, T * H * 18)           # y and x read and written, the normed row written
+        out["rows_begin"] = (0.0, False, T * H * 10)           # x read, y cleared, the normed row written
         out["rmsnorm"] = (0.0, False, T * H * 6)
         by = {l["type"]: l["mixer"] for l in cfg["layers"]}
         if "mamba1" in by:
