@@ -4,6 +4,7 @@ projection kernel, its results saved with torch.save to the path given as the on
 
   * Tiny A in bfloat16: four prompts of unequal lengths in one step, then eight tokens each;
   * a Botulorn model of four layers with latent attention (one-token steps over cached rows) likewise;
+  * a Gidurax model with every kind of layer and a run that repeats (all experts chosen: no choice hangs on rounding);
   * two layers at 7B sizes in bfloat16: a 300-token prompt whole, then three requests batched,
     their last 32 / 5 / 17 tokens one by one (split-K projections, decode attention over
     several pages, a window of 160 that cuts the longest request);
@@ -20,15 +21,21 @@ sys.path.insert(0, os.path.dirname(TESTS))
 sys.path.insert(0, TESTS)
 
 from helpers import TINY_A, prompts_for                                 # noqa: E402
+import test_gpu_gidurax as G                                            # noqa: E402
 from test_gpu_botulorn import TENSOR                                    # noqa: E402
 from test_gpu_full_size import CFG, LENGTHS, run_batched_with_tails     # noqa: E402
+
+SANDWICH = G.config([G.layer(G.scan(inner=256, state=16, dt_rank=16), G.dense(256)),
+                     G.layer(G.delta(heads=4, kv_heads=2, dim=64, vdim=32), G.moe(ff=64, experts=4, top=5, identity=1, shared=64)),
+                     G.layer(G.attn(heads=8, kv_heads=2, dim=64, vdim=48, scale=0.3), None)], width=128, vocab=160, loop=(1, 3, 2))
 
 
 def main(path: str) -> None:
     from inference_engine_rust_b200 import LoadedModel
     from inference_engine_rust_b200.csrc import bindings as B
     out = {}
-    for name, cfg, vocab in (("tiny", dict(TINY_A), TINY_A["vocab_size"]), ("latent", TENSOR, TENSOR["vocab"])):
+    for name, cfg, vocab in (("tiny", dict(TINY_A), TINY_A["vocab_size"]), ("latent", TENSOR, TENSOR["vocab"]),
+                             ("sandwich", SANDWICH, SANDWICH["vocab"])):
         tiny = LoadedModel.random(cfg, seed=3, dtype="bfloat16", std=0.1)
         eng = tiny.session(max_tokens=64 * 8, poison_cache=True).engine
         prompts = prompts_for({"vocab_size": vocab}, [5, 11, 23, 70], seed=2)

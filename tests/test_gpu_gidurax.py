@@ -601,7 +601,7 @@ def test_one_far_key_decides(root, n, place, dtype):
 
 
 def _remembering(t):
-    """States that hardly decay, written strongly by token 48 alone (its row is large, so its gates and values are)."""
+    """States that hardly decay."""
     for n in t:
         if n.endswith("dt.b") or n.endswith("dt_bias"):
             t[n] = torch.full_like(t[n], -9.0)

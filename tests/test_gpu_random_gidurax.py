@@ -19,7 +19,7 @@ def draw_mixer(rng):
     kind = rng.choice(["delta", "attention", "mamba1"])
     kv, group = rng.choice([1, 2, 3, 4]), rng.choice([1, 2, 3])
     if kind == "delta":
-        return T.delta(heads=kv * group, kv_heads=kv, dim=rng.choice([8, 16, 32, 64]), vdim=rng.choice([7, 16, 24, 32, 64, 96]), conv=rng.choice([1, 2, 3, 4, 6]))
+        return T.delta(heads=kv * group, kv_heads=kv, dim=rng.choice([16, 24, 32, 64]), vdim=rng.choice([7, 16, 24, 32, 64, 96]), conv=rng.choice([1, 2, 3, 4, 6]))
     if kind == "attention":
         dim = rng.choice([4, 8, 16, 24, 32, 48, 64, 80, 128])
         return T.attn(heads=kv * group, kv_heads=kv, dim=dim, vdim=rng.choice([dim, 8, 20, 48, 64]), scale=round(dim ** -0.5 * rng.choice([0.5, 1.0]), 4),
@@ -78,5 +78,10 @@ def test_random_configuration(root, case):
                 eng.close_sequence(slots[i])
                 live.remove(i)
         eng.check_device()
-        for i in range(len(prompts)):
-            T.compare(torch.cat(rows[i]), want[i], dtype, f"case {case} ({dtype}), request {i}: {cfg}", slack=max(1.0, runs / 3))
+        for i, p in enumerate(prompts):
+            slack = max(1.0, runs / 3)
+            if dtype == "bfloat16":         # how far rounding alone moves this model (a read-out near zero under a norm moves far)
+                exact = P.forward(cfg, weights, p)
+                noise = ((exact - want[i]).pow(2).mean(-1).sqrt() / exact.abs().max()).max().item()
+                slack = max(slack, 1.5 * noise / 0.012)
+            T.compare(torch.cat(rows[i]), want[i], dtype, f"case {case} ({dtype}), request {i}: {cfg}", slack=slack)
